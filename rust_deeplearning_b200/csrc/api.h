@@ -11,7 +11,7 @@ extern "C" {
 #define RDL_ACT_SILU 1
 #define RDL_ACT_SWISH_LIMIT 2   // min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1), L a parameter
 
-#define RDL_ABI_VERSION 19
+#define RDL_ABI_VERSION 20
 
 const char* rdl_last_error(void);
 int rdl_abi_version(void);
@@ -22,6 +22,7 @@ void rdl_set_programmatic_launch(int on);
 // Codes a kernel leaves in the step's status word (an int the host reads after the step).  Each
 // kernel that can give up a bounded wait has its own.
 #define RDL_FAULT_TOKEN_ID 1           // embed_rows: a token id outside the table (its row is NaN)
+#define RDL_FAULT_POSITION 2           // embed_rows: a position beyond the position table (its row is NaN)
 #define RDL_FAULT_ATTENTION_DECODE 3   // attention_decode: a page copy did not complete
 #define RDL_FAULT_GEMM_TC 4            // gemm_tc, one block a tile: a stage or an accumulator was not handed over
 #define RDL_FAULT_ATTENTION_TC 5       // attention_prefill_tc: a tile copy or a product did not complete
@@ -70,6 +71,13 @@ typedef struct {
     // optional: one float per query head; the weight of a visible key is then sigmoid(score + sigmoid_bias[h]) and
     // the weights are not normalised over the keys (no softmax, no denominator, no sinks); NULL: softmax
     const float* sigmoid_bias;
+    // optional: chunk > 0 - positions form chunks of so many, counted from the sequence's start, and a query sees the keys
+    // of its own chunk only (beside the causal rule and the window)
+    int chunk;
+    // optional: [n_heads][rel_len] floats added to the scaled (and capped) scores by head and distance p - j (the last
+    // entry stands for every larger distance); NULL: none.  rdl_attention_plain takes it as it is, the bfloat16 kernels
+    // (prefill, prefill_tc, decode) take it times log2(e)
+    const float* rel_bias; int rel_len;
     // filled in by the launcher: clock cycles after which a wait is given up, and the test's extra bytes
     long long wait_cycles; int test_extra_tx;
 } AttentionArgs;
@@ -83,13 +91,15 @@ int rdl_attention_prefill_tc(const AttentionArgs* a, long long row_width, void* 
 long long rdl_attention_decode_counter_bytes(int n_tokens, int n_kv_heads);
 long long rdl_attention_decode_scratch_bytes(int n_tokens, int n_heads, int n_kv_heads, int head_dim, int max_splits);
 
+// out[t] = table[ids[t]] * scale (+ pos_table[tok_pos[t]] if pos_table [n_pos][hidden] is given; a position below 0 adds nothing)
 int rdl_embed_rows(void* out_f32, const void* table, int table_dtype, const int* ids, float scale,
-                   int n_rows, int hidden, int vocab, int* status, void* stream);
+                   int n_rows, int hidden, int vocab, int* status, const void* pos_table, int pos_dtype,
+                   const int* tok_pos, int n_pos, void* stream);
 int rdl_norm_residual_norm(const void* x, int x_dtype, const int* row_index,
                            const void* w1, int w1_dtype, float eps1, float off1, void* res_f32,
                            const void* w2, int w2_dtype, float eps2, float off2,
                            void* y, int y_dtype, int n_rows, int hidden, void* stream);
-int rdl_gated_activation(void* out, const void* gate_up, int dtype, int activation, int n_rows, int inter, void* stream);
+int rdl_gated_activation(void* out, const void* gate_up, int dtype, int activation, int n_rows, int inter, float act_param, void* stream);
 int rdl_softcap_inplace(void* z_f32, long long total, float cap, void* stream);
 int rdl_scale_inplace(void* z_f32, long long total, float scale, void* stream);
 int rdl_residual_add(void* res_f32, const void* x, int x_dtype, long long total, void* stream);
@@ -131,6 +141,42 @@ int rdl_rope_projnorm_cache(void* rows, long long row_stride, int dtype, int n_t
                             int do_rope, const float* wq, const float* wk, float eps, int q_count, int k_count, int do_write,
                             void* k_cache, void* v_cache, const int* tables, int table_width, int page_size, int ring_pages,
                             const int* seq_end, void* stream);
+
+// ---- short convolution, projection norms, value mixing and cache write (csrc/qkv_prepare.cu) ----
+// The packed rows of a q/k/v product ([tokens][n_heads query, n_kv_heads key, n_kv_heads value heads of head_dim]) made ready
+// for attention, into another buffer of packed rows and into the cache; every mechanism is optional (NULL: left out).
+typedef struct {
+    int dtype;                                  // of rows, out, conv, v_first and the cache
+    int n_tokens, n_seqs, n_heads, n_kv_heads, head_dim;
+    const void* rows; long long row_stride;
+    void* out; long long out_stride;
+    const float* bias;                          // [channels], added to the projection
+    const void* conv; int taps;                 // [taps][channels]: weight j multiplies the value taps - 1 - j tokens back
+    float* state;                               // [slots][taps - 1][channels], the last values of rows + bias
+    const float* wq; const float* wk;           // [n_heads * head_dim], [n_kv_heads * head_dim]
+    float eps, q_count, k_count;
+    const void* v_first; long long v_first_stride; float v_lambda;      // v <- (1 - v_lambda) v + v_lambda v_first
+    const int* tok_seq; const int* tok_pos; const int* seq_start; const int* slots; const int* seq_end;
+    int do_write;
+    void* k_cache; void* v_cache; const int* tables; int table_width, page_size, ring_pages;
+    int n_channels;                             // filled in by the launcher
+} QkvPrepareArgs;
+int rdl_qkv_prepare(const QkvPrepareArgs* a, void* stream);
+
+// ---- hyper-connections: a residual stream of several copies (csrc/hyper.cu) ----
+typedef struct {
+    int n_rows, width, n_copies, in_copies;     // in_copies 1: x_in is one row that stands for all copies
+    const float* x_in;                          // [rows][in_copies][width]
+    float* x_out;                               // [rows][n_copies][width], optional; may be x_in where in_copies == n_copies
+    const void* a; const void* b; int branch_dtype;      // the sublayer's result y = a + b * sigmoid(b_gate[row * gate_stride])
+    const float* b_gate; long long gate_stride;          // optional (b then counts whole)
+    const float* mix; const float* write;       // [n_copies from][n_copies to], [n_copies]
+    const float* read;                          // [n_copies]
+    const void* w; int w_dtype; float eps, off; // the norm of the weighted sum; NULL: the sum itself
+    void* out; int out_dtype;                   // [rows][width], optional
+    const int* row_index;                       // optional: output row r is row row_index[r] (x_out must then be NULL)
+} HyperArgs;
+int rdl_hyper(const HyperArgs* a, void* stream);
 
 // ---- forms of the residual stream and of gates (csrc/rownorm.cu) ----
 // Norm after the sum: res <- norm(alpha * res + branch) with norm(v) = v / sqrt(mean(v^2) + eps) * (w + off), in float;
@@ -245,11 +291,12 @@ int rdl_decay_attention_chunked(const DecayAttentionArgs* a, void* work, long lo
 int rdl_gemm_f32(void* out, const void* x, const void* w, int m, int n, int k, void* stream);
 
 // out[m, n] = epilogue(sum_k x[m, k] * w[n, k]) for m <= 16, bfloat16 operands, float accumulation.
-// gated: w is [2 n, k] (gate rows, then up rows) and the result is act(gate) * up.
+// gated: w is [2 n, k] (gate rows, then up rows) and the result is act(gate) * up (or a gated form with a parameter,
+// act_param).
 // softcap > 0: cap * tanh(v / cap).  out_dtype: RDL_F32 or RDL_BF16.  status (optional) is set non-zero
 // when a block gives up a bounded wait for a copy.
 int rdl_gemm_skinny(void* out, int out_dtype, const void* x, const void* w, int m, int n, int k,
-                    int gated, int activation, float softcap, int* status, void* stream);
+                    int gated, int activation, float softcap, int* status, float act_param, void* stream);
 
 // The norms around a few-row product taken off the step's critical path ("deferred norms").
 // A branch of the residual stream h ends in a product P (up to 8 rows, as many columns as the stream is wide)
@@ -289,7 +336,8 @@ typedef struct {
 // rdl_gemm_skinny with m <= 8 and one side of a deferred norm.  P: plain epilogue only (not gated, no soft-cap),
 // `out` unused.  C: any epilogue; m counts the rows of each half of the operand.
 int rdl_gemm_skinny_norm(void* out, int out_dtype, const void* x, const void* w, int m, int n, int k,
-                         int gated, int activation, float softcap, const DeferredNormArgs* norm, int* status, void* stream);
+                         int gated, int activation, float softcap, const DeferredNormArgs* norm, int* status, float act_param,
+                         void* stream);
 // Rows of a residual stream outside a product: h' = h + s1 a' with s1 from the sums (sums NULL: h' = h), written
 // to residual_out (optional; may be residual_in), and scaled = h' (w + off) as bfloat16 (optional).
 int rdl_stream_rows(const float* sums, int n_sums, float eps1, const void* branch, const float* residual_in,
@@ -300,7 +348,7 @@ int rdl_stream_rows(const float* sums, int n_sums, float eps1, const void* branc
 // tensor memory).  n must be a positive number, k a multiple of 8; status (optional) is set non-zero
 // when a block gives up a bounded wait.
 int rdl_gemm_tc(void* out, int out_dtype, const void* x, const void* w, int m, int n, int k,
-                int gated, int activation, float softcap, int* status, void* stream);
+                int gated, int activation, float softcap, int* status, float act_param, void* stream);
 
 // ---- latent attention (csrc/latent.cu) ----
 // One call per layer run and step: rotates the rotated part of every query head (in place, or into
@@ -361,10 +409,15 @@ int rdl_latent_decode(void* out, long long out_stride, const void* q, long long 
 #define RDL_ROUTE_SOFTMAX 0
 // RDL_ROUTE_SOFTMAX_CHOSEN: the choice is by the logits themselves and the weights are the softmax over the chosen
 // logits only.  bias (optional, float [experts]) is added to the logits before anything else, in every form.
+// extra: so many rows of w_router beyond the experts' only form logits (logits is [rows][experts + extra]).
+// n_groups > 0: the experts form so many equal groups of neighbours, a group's score is the sum of its two largest choices,
+// and only experts of the `keep` best groups can be chosen.  norm_eps > 0: the chosen scores are divided by (their sum +
+// norm_eps) (not with RDL_ROUTE_SOFTMAX_CHOSEN).
 #define RDL_ROUTE_SIGMOID 1
 #define RDL_ROUTE_SOFTMAX_CHOSEN 2
 int rdl_moe_route(const void* x, int dtype, const float* w_router, const float* bias, const float* correction, int n_rows,
-                  int n_experts, int width, int top, int scoring, int* sel, float* sel_w, float* logits, void* stream);
+                  int n_experts, int width, int top, int scoring, int* sel, float* sel_w, float* logits, int extra, int n_groups,
+                  int keep, float norm_eps, void* stream);
 // mid[(t, k), :] = gated(W_gate[e] x_t, W_up[e] x_t) for e = sel[t, k] < n_real; w_gate_up [n_real][2 ff][width]
 // activation >= 16 (RDL_UNARY_*): experts of two matrices, mid = act(W_up[e] x_t) with w_gate_up [n_real][ff][width].
 // sel_w (optional): the pair's weight multiplies the expert's input, mid = f(W (sel_w[t, k] x_t)).

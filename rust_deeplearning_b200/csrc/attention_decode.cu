@@ -63,8 +63,6 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-__host__ __device__ inline int first_key(int p, int window) { return window > 0 ? (p - window + 1 > 0 ? p - window + 1 : 0) : 0; }
-
 __device__ __forceinline__ void mbar_init(uint32_t bar, int count) {
     asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count));
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -107,7 +105,8 @@ __device__ __forceinline__ bool mbar_wait_bounded(uint32_t bar, uint32_t parity,
 // HD: head_dim padded to 64, 128 or 256 (head_dim itself is a multiple of 16).  EXACT: head_dim == HD;
 // row sizes and the swizzle are then compile-time constants and a fragment's address is a register
 // plus an immediate.
-template <int HD, bool EXACT, bool SIG>
+// MODE 0: softmax; 1: sigmoid weights; 2: softmax with a bias per head and distance (base-2 domain) added to the scores.
+template <int HD, bool EXACT, int MODE>
 __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(AttentionArgs a) {
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ __align__(8) unsigned long long bar_storage[3];     // one per tile of the ring
@@ -130,7 +129,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     }
     const int seq = a.tok_seq[t], p = a.tok_pos[t];
     if (p < 0) return;  // a padding row of a fixed-size batch
-    const int lo = first_key(p, a.window);
+    const int lo = rdl_first_key(p, a.window, a.chunk);
     const int split0 = lo / a.keys_per_split;
     const int n_splits = p / a.keys_per_split - split0 + 1;
     if (sp >= n_splits) return;
@@ -195,7 +194,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     // With new_rows no other kernel writes the cache in this step: every first page is fetched early.
     const bool fuse = a.new_rows != 0;
     const bool early = fuse || (a.seq_past != nullptr && (page_first + 1) * ps <= a.seq_past[seq] &&
-                                (a.window <= 0 || t == a.seq_start[seq + 1] - 1));
+                                ((a.window <= 0 && a.chunk <= 0) || t == a.seq_start[seq + 1] - 1));
     if (early && tid == 0) {
         issue(0);
         issue(1);
@@ -274,7 +273,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     // Sigmoid weights (no softmax): the weight of a key is sigmoid(score + bias[h]) by itself, so nothing is rescaled and
     // nothing is divided in the end.  The merges below stay as they are: every maximum is 0 (all their weights are 1) and
     // the normaliser is replaced by 1.  The weights reach the tensor cores as two bfloat16 terms (16 bits of them count).
-    constexpr bool sig = SIG;
+    constexpr bool sig = MODE == 1;
     float sb0 = 0.f, sb1 = 0.f;
     if (sig) {
         m0 = m1 = 0.f;
@@ -284,6 +283,9 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     const bool capped = a.softcap > 0.f;
     const float c_in = capped ? a.score_scale / a.softcap : a.score_scale * LOG2E;
     const float c_out = a.softcap * LOG2E;
+    // the bias tables of heads 2 tq and 2 tq + 1 (a column beyond the group's heads reads its first head's)
+    const float* rel0 = MODE == 2 ? a.rel_bias + (long long)(g * G + (2 * tq < G ? 2 * tq : 0)) * a.rel_len : nullptr;
+    const float* rel1 = MODE == 2 ? a.rel_bias + (long long)(g * G + (2 * tq + 1 < G ? 2 * tq + 1 : 0)) * a.rel_len : nullptr;
 
     // Fragment addresses.  Keys (A of the score product): row w0 + (lane & 15), chunk 2 kk + (lane >> 4).
     // Values (A of the output product, transposed on load): row w0 + (lane & 7) + 8 (lane >> 4), chunk
@@ -361,6 +363,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
             for (int e = 0; e < 4; ++e) {
                 float v = capped ? tanh_fast(s[e] * c_in) * c_out : s[e] * c_in;
                 const int r = w0 + quad + 8 * (e >> 1);
+                if (MODE == 2) v += __ldg(((e & 1) ? rel1 : rel0) + min(max(p - (lp * ps + r), 0), a.rel_len - 1));
                 if (r < r_begin || r >= r_end) v = -INFINITY;
                 s[e] = v;
             }
@@ -590,7 +593,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     }
 }
 
-template <int HD, bool EXACT, bool SIG>
+template <int HD, bool EXACT, int MODE>
 int launch_decode_as(const AttentionArgs* a, cudaStream_t st) {
     const int tiles = 3 * a->page_size * a->head_dim * 2;
     const int merge = DEC_WARPS * QROWS * HD * (int)sizeof(float);
@@ -601,7 +604,7 @@ int launch_decode_as(const AttentionArgs* a, cudaStream_t st) {
                 a->page_size, a->head_dim, smem);
     static int granted = 32 * 1024;      // above this the kernel (which also has a few KB of static shared memory) opts in
     if (smem > granted) {
-        RDL_CUDA(cudaFuncSetAttribute(attention_decode_kernel<HD, EXACT, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem),
+        RDL_CUDA(cudaFuncSetAttribute(attention_decode_kernel<HD, EXACT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem),
                  "attention_decode");
         granted = smem;
     }
@@ -609,14 +612,15 @@ int launch_decode_as(const AttentionArgs* a, cudaStream_t st) {
     AttentionArgs b = *a;
     b.wait_cycles = rdl_wait_cycles_for(RDL_FAULT_ATTENTION_DECODE);
     b.test_extra_tx = rdl_test_extra_tx_for(RDL_FAULT_ATTENTION_DECODE);
-    RDL_CHECK_EX(rdl_launch(attention_decode_kernel<HD, EXACT, SIG>, grid, dim3(DEC_THREADS), (size_t)smem, st, b), "attention_decode");
+    RDL_CHECK_EX(rdl_launch(attention_decode_kernel<HD, EXACT, MODE>, grid, dim3(DEC_THREADS), (size_t)smem, st, b), "attention_decode");
     return 0;
 }
 
-// softmax, or sigmoid weights (a kernel of their own, so that the softmax kernels keep their registers)
+// softmax, sigmoid weights or a distance bias (kernels of their own, so that the softmax kernels keep their registers)
 template <int HD, bool EXACT>
 int launch_decode(const AttentionArgs* a, cudaStream_t st) {
-    return a->sigmoid_bias ? launch_decode_as<HD, EXACT, true>(a, st) : launch_decode_as<HD, EXACT, false>(a, st);
+    return a->sigmoid_bias ? launch_decode_as<HD, EXACT, 1>(a, st)
+                           : (a->rel_bias ? launch_decode_as<HD, EXACT, 2>(a, st) : launch_decode_as<HD, EXACT, 0>(a, st));
 }
 
 }  // namespace

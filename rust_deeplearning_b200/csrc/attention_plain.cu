@@ -8,6 +8,7 @@
 //   s_j = (q_h . k_g,j) * score_scale                    attention.rs:413-416
 //   s_j = cap * tanh(s_j / cap)            if cap > 0    attention.rs:419-423
 //   keys kept: j <= p and (window == 0 or p - j < window)  ops.rs:905-922, :932-952
+//   (with chunk: j / chunk == p / chunk as well; with rel_bias: s_j += rel_bias[h][min(p - j, rel_len - 1)]; the reference has neither)
 //   a = softmax_j(s)                                      ops.rs:598-608
 //   (with sinks: the denominator also holds exp(sinks[h]); the reference has none)
 //   (with sigmoid_bias: a_j = sigmoid(s_j + sigmoid_bias[h]) for the keys kept, not normalised; the reference has none)
@@ -37,7 +38,8 @@ __global__ void attention_plain_kernel(AttentionArgs a) {
     const int new_row0 = a.seq_start[seq] - a.seq_past[seq];  // packed row of position j is new_row0 + j
     const int* table = a.tables ? a.tables + (long long)seq * a.table_width : nullptr;
     const T* q = (const T*)a.q + (long long)t * a.q_stride + (long long)h * hd;
-    const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+    const int lo = rdl_first_key(p, a.window, a.chunk);
+    const float* rel = a.rel_bias ? a.rel_bias + (long long)h * a.rel_len : nullptr;
 
     float acc[CHUNKS];
 #pragma unroll
@@ -68,6 +70,7 @@ __global__ void attention_plain_kernel(AttentionArgs a) {
             for (int i = 0; i < hd; ++i) d = fmaf(to_float(q[i]), to_float(kp[sw < 0 ? i : rdl_cache_col<T>(sw, i, hd)]), d);
             d *= a.score_scale;
             if (a.softcap > 0.f) d = a.softcap * tanhf(d / a.softcap);
+            if (rel) d += rel[min(p - j, a.rel_len - 1)];
             s = d;
         }
         float pj;
@@ -122,7 +125,9 @@ int rdl_check_attention_args(const AttentionArgs* a, const char* who) {
     RDL_REQUIRE(a->n_heads > 0 && a->n_kv_heads > 0 && a->n_heads % a->n_kv_heads == 0,
                 "%s: %d heads cannot share %d key/value heads", who, a->n_heads, a->n_kv_heads);
     RDL_REQUIRE(a->head_dim > 0, "%s: bad head_dim %d", who, a->head_dim);
-    RDL_REQUIRE(a->window >= 0 && a->softcap >= 0.f, "%s: window and soft-cap must not be negative", who);
+    RDL_REQUIRE(a->window >= 0 && a->chunk >= 0 && a->softcap >= 0.f, "%s: window, chunk and soft-cap must not be negative", who);
+    RDL_REQUIRE(!a->rel_bias || a->rel_len > 0, "%s: a distance bias needs at least one entry a head", who);
+    RDL_REQUIRE(!(a->rel_bias && a->sigmoid_bias), "%s: sigmoid weights come without a distance bias", who);
     RDL_REQUIRE(a->q && a->out && a->tok_seq && a->tok_pos && a->seq_start && a->seq_past && a->seq_cached,
                 "%s: missing query, output or batch description", who);
     RDL_REQUIRE(a->q_stride >= (long long)a->n_heads * a->head_dim && a->out_stride >= (long long)a->n_heads * a->head_dim,

@@ -50,7 +50,8 @@ __device__ __forceinline__ uint32_t tile_addr(uint32_t base, int row, int chunk)
     return base + (uint32_t)((row * (HD / 8) + swizzled_chunk<HD>(row, chunk)) * 16);
 }
 
-template <int HD, bool SIG>
+// MODE 0: softmax; 1: sigmoid weights; 2: softmax with a bias per head and distance (base-2 domain) added to the scores
+template <int HD, int MODE>
 __global__ void __launch_bounds__(NTHREADS) attention_prefill_kernel(AttentionArgs a) {
     constexpr int CH = HD / 8;          // 16-byte chunks per row
     extern __shared__ __align__(128) unsigned char smem[];
@@ -90,20 +91,23 @@ __global__ void __launch_bounds__(NTHREADS) attention_prefill_kernel(AttentionAr
     }
 
     const int p_first = past + q0, p_last = past + q0 + rows - 1;
-    const int lo_first = a.window > 0 ? max(0, p_first - a.window + 1) : 0;
+    const int lo_first = rdl_first_key(p_first, a.window, a.chunk);
     // positions of the two rows this thread holds
     const int pr0 = p_first + warp * 16 + quad, pr1 = pr0 + 8;
     const int pw_first = p_first + warp * 16, pw_last = pw_first + 15;
+    const int lo0 = rdl_first_key(pr0, a.window, a.chunk), lo1 = rdl_first_key(pr1, a.window, a.chunk);
+    const int low_first = rdl_first_key(pw_first, a.window, a.chunk), low_last = rdl_first_key(pw_last, a.window, a.chunk);
 
     float o[HD / 8][4];
 #pragma unroll
     for (int i = 0; i < HD / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     const float LOG2E = 1.4426950408889634f;
-    constexpr bool sig = SIG;                                             // weights sigmoid(score + bias[h]), not normalised
+    constexpr bool sig = MODE == 1;                                             // weights sigmoid(score + bias[h]), not normalised
     const float sig_bias = sig ? a.sigmoid_bias[h] * LOG2E : 0.f;         // in the base-2 domain, like the scores
     const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
     const int ksteps = (hd + 15) / 16;
+    const float* rel = MODE == 2 ? a.rel_bias + (long long)h * a.rel_len : nullptr;      // entry n: distance n, the last one for all beyond
 
     // One tile of keys (which == 0) or values (which == 1) on its way to shared memory: asynchronous
     // 16-byte copies that bypass the registers, rows beyond the sequence and chunks beyond head_dim
@@ -141,7 +145,7 @@ __global__ void __launch_bounds__(NTHREADS) attention_prefill_kernel(AttentionAr
         __syncthreads();
 
         // this warp's rows see nothing of the tile: skip its arithmetic (barriers stay outside)
-        const bool warp_active = kv0 <= pw_last && (a.window == 0 || pw_first - (kv0 + BN - 1) < a.window);
+        const bool warp_active = kv0 <= pw_last && kv0 + BN - 1 >= low_first;
         uint32_t pf[BN / 16][4];
         uint32_t pl[BN / 16][4];      // sigmoid weights: what the rounding of pf left
         if (warp_active) {
@@ -161,7 +165,8 @@ __global__ void __launch_bounds__(NTHREADS) attention_prefill_kernel(AttentionAr
                 }
             }
             // ---- scale, soft-cap, mask ----
-            const bool need_mask = !(kv0 + BN - 1 <= pw_first && (a.window == 0 || pw_last - kv0 < a.window));
+            const bool need_mask = !(kv0 + BN - 1 <= pw_first && kv0 >= low_last);
+            const bool rel_plain = MODE == 2 && kv0 + BN - 1 <= pw_first && pw_last - kv0 < a.rel_len;     // every distance of the tile has an entry
             float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
             for (int nt = 0; nt < BN / 8; ++nt) {
@@ -169,11 +174,15 @@ __global__ void __launch_bounds__(NTHREADS) attention_prefill_kernel(AttentionAr
                 for (int e = 0; e < 4; ++e) {
                     float v = s[nt][e] * a.score_scale;
                     if (a.softcap > 0.f) v = a.softcap * tanh_fast(v * inv_cap);
-                    v *= LOG2E;
+                    if (MODE == 2) {
+                        const int dist = ((e < 2) ? pr0 : pr1) - (kv0 + nt * 8 + 2 * tq + (e & 1));
+                        v = fmaf(v, LOG2E, __ldg(rel + (rel_plain ? dist : min(max(dist, 0), a.rel_len - 1))));
+                    } else {
+                        v *= LOG2E;
+                    }
                     if (need_mask) {
                         const int key = kv0 + nt * 8 + 2 * tq + (e & 1);
-                        const int pr = (e < 2) ? pr0 : pr1;
-                        const bool keep = key <= pr && (a.window == 0 || pr - key < a.window);
+                        const bool keep = key <= ((e < 2) ? pr0 : pr1) && key >= ((e < 2) ? lo0 : lo1);
                         if (!keep) v = -INFINITY;
                     }
                     s[nt][e] = v;
@@ -279,24 +288,24 @@ __global__ void __launch_bounds__(NTHREADS) attention_prefill_kernel(AttentionAr
     }
 }
 
-template <int HD, bool SIG>
+template <int HD, int MODE>
 int launch_prefill_as(const AttentionArgs* a, cudaStream_t st) {
     const int smem = (BM + 2 * BN) * HD * 2;
     static bool opted = false;
     if (smem > 48 * 1024 && !opted) {
-        RDL_CUDA(cudaFuncSetAttribute(attention_prefill_kernel<HD, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem),
+        RDL_CUDA(cudaFuncSetAttribute(attention_prefill_kernel<HD, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem),
                  "attention_prefill");
         opted = true;
     }
     dim3 grid(a->n_tiles, a->n_heads);
-    RDL_CHECK_EX(rdl_launch(attention_prefill_kernel<HD, SIG>, grid, dim3(NTHREADS), (size_t)smem, st, *a), "attention_prefill");
+    RDL_CHECK_EX(rdl_launch(attention_prefill_kernel<HD, MODE>, grid, dim3(NTHREADS), (size_t)smem, st, *a), "attention_prefill");
     return 0;
 }
 
-// softmax, or sigmoid weights (a kernel of their own, so that the softmax kernels keep their registers)
+// softmax, sigmoid weights or a distance bias (kernels of their own, so that the softmax kernels keep their registers)
 template <int HD>
 int launch_prefill(const AttentionArgs* a, cudaStream_t st) {
-    return a->sigmoid_bias ? launch_prefill_as<HD, true>(a, st) : launch_prefill_as<HD, false>(a, st);
+    return a->sigmoid_bias ? launch_prefill_as<HD, 1>(a, st) : (a->rel_bias ? launch_prefill_as<HD, 2>(a, st) : launch_prefill_as<HD, 0>(a, st));
 }
 
 }  // namespace

@@ -117,10 +117,13 @@ struct TcAttnArgs {
     int window;
     int* status;
     const float* sinks;
+    int chunk;
+    const float* rel_bias; int rel_len;      // [n_heads][rel_len] in the base-2 domain; NULL: none
+    int rel_in_smem;                         // the head's table fits beside the tiles
 };
 
-// DB: 64-column blocks of a head (head_dim / 64)
-template <int DB>
+// DB: 64-column blocks of a head (head_dim / 64).  REL: a bias per head and distance is added to the scores.
+template <int DB, bool REL>
 __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                       const __grid_constant__ CUtensorMap map_kv, TcAttnArgs a) {
     // 64-row tiles come from the host; a block takes two of them, so odd ones have nothing to do
@@ -144,6 +147,7 @@ __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __gr
     unsigned char* sK = sQ + q_bytes;                  // two stages
     unsigned char* sV = sK + 2 * kv_bytes;             // two stages
     unsigned char* sP = sV + 2 * kv_bytes;             // [128 rows][128 bytes]
+    float* sRel = reinterpret_cast<float*>(sP + QM * 128);      // [rel_len], where it fits
     __shared__ __align__(8) unsigned long long q_full, k_full[2], v_full[2], k_empty[2], v_empty[2], s_full, s_empty, p_full, pv_done;
     __shared__ uint32_t tmem_slot;
     const uint32_t tmem_cols = hd <= 64 ? 128 : (hd <= 192 ? 256 : 512);   // 64 for S, head_dim for O, a power of two
@@ -162,6 +166,11 @@ __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __gr
         mbar_init(smem_u32(&pv_done), 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
+    const float* rel = REL ? a.rel_bias + (long long)h * a.rel_len : nullptr;
+    if (REL && a.rel_in_smem) {          // a constant of the model: copied while the kernel before is still running
+        for (int i = threadIdx.x; i < a.rel_len; i += ATC_THREADS) sRel[i] = __ldg(rel + i);
+        rel = sRel;
+    }
     if (warp == 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_slot)), "r"(tmem_cols) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
@@ -176,7 +185,7 @@ __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __gr
 
     // the tiles of keys this block visits: positions [kv_first, p_last], 64 at a time
     const int p_first = q0, p_last = q0 + rows - 1;
-    const int lo_first = a.window > 0 ? max(0, p_first - a.window + 1) : 0;
+    const int lo_first = rdl_first_key(p_first, a.window, a.chunk);
     const int kv_first = (lo_first / KN) * KN;
     const int n_kv = (p_last - kv_first) / KN + 1;
     bool ok = true;
@@ -269,6 +278,7 @@ __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __gr
         const float c_in = capped ? a.score_scale / a.softcap : a.score_scale * LOG2E;
         const float c_out = a.softcap * LOG2E;
         const int pr_warp_first = q0 + q * 32, pr_warp_last = pr_warp_first + 31;
+        const int pr_lo = rdl_first_key(pr, a.window, a.chunk), lo_warp_last = rdl_first_key(pr_warp_last, a.window, a.chunk);
         float m_ref = -INFINITY, l = 0.f;
         for (int j = 0; j < n_kv && ok; ++j) {
             if (!mbar_wait_bounded(smem_u32(&s_full), j & 1)) { ok = false; break; }
@@ -290,14 +300,25 @@ __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __gr
             if (capped) {
 #pragma unroll
                 for (int i = 0; i < KN; ++i) t[i] = tanh_fast(t[i] * c_in) * c_out;
-            } else {
+            } else if (!REL) {
 #pragma unroll
                 for (int i = 0; i < KN; ++i) t[i] *= c_in;
             }
+            if (REL) {
+                const float c = capped ? 1.0f : c_in;
+                if (key0 + KN - 1 <= pr_warp_first && pr_warp_last - key0 < a.rel_len) {      // every distance has an entry
+                    const float* rp = rel + (pr - key0);
+#pragma unroll
+                    for (int i = 0; i < KN; ++i) t[i] = fmaf(t[i], c, rp[-i]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < KN; ++i) t[i] = fmaf(t[i], c, rel[min(max(pr - key0 - i, 0), a.rel_len - 1)]);
+                }
+            }
             // tiles that every row of this warp sees whole need no masks (the test is the same for all lanes)
-            const bool interior = key0 + KN - 1 <= pr_warp_first && (a.window == 0 || pr_warp_last - key0 < a.window);
+            const bool interior = key0 + KN - 1 <= pr_warp_first && key0 >= lo_warp_last;
             if (!interior) {
-                const int hi = pr - key0, lo = a.window > 0 ? pr - a.window + 1 - key0 : -1;   // tile columns [lo, hi] are visible
+                const int hi = pr - key0, lo = pr_lo - key0;   // tile columns [lo, hi] are visible
 #pragma unroll
                 for (int i = 0; i < KN; ++i)
                     if (i > hi || i < lo) t[i] = -INFINITY;
@@ -420,15 +441,20 @@ int make_map(CUtensorMap* map, const void* ptr, long long rows, long long cols, 
     return 0;
 }
 
+template <int DB, bool REL>
+int launch_tc_as(dim3 grid, int smem, cudaStream_t st, const CUtensorMap& map_q, const CUtensorMap& map_kv, const TcAttnArgs& t) {
+    static int granted = 0;
+    if (smem > granted) {
+        RDL_CUDA(cudaFuncSetAttribute(attention_tc_kernel<DB, REL>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "attention_prefill_tc");
+        granted = smem;
+    }
+    RDL_CHECK_EX(rdl_launch(attention_tc_kernel<DB, REL>, grid, dim3(ATC_THREADS), (size_t)smem, st, map_q, map_kv, t), "attention_prefill_tc");
+    return 0;
+}
+
 template <int DB>
 int launch_tc(dim3 grid, int smem, cudaStream_t st, const CUtensorMap& map_q, const CUtensorMap& map_kv, const TcAttnArgs& t) {
-    static bool opted = false;
-    if (!opted) {
-        RDL_CUDA(cudaFuncSetAttribute(attention_tc_kernel<DB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "attention_prefill_tc");
-        opted = true;
-    }
-    RDL_CHECK_EX(rdl_launch(attention_tc_kernel<DB>, grid, dim3(ATC_THREADS), (size_t)smem, st, map_q, map_kv, t), "attention_prefill_tc");
-    return 0;
+    return t.rel_bias ? launch_tc_as<DB, true>(grid, smem, st, map_q, map_kv, t) : launch_tc_as<DB, false>(grid, smem, st, map_q, map_kv, t);
 }
 
 }  // namespace
@@ -454,8 +480,17 @@ extern "C" int rdl_attention_prefill_tc(const AttentionArgs* a, long long row_wi
     if (int e = make_map(&map_q, a->q, a->n_tokens, row_width, QM)) return e;
     if (int e = make_map(&map_kv, a->q, a->n_tokens, row_width, KN)) return e;
     TcAttnArgs t{a->out, a->out_stride, a->tile_seq, a->tile_q0, a->n_tiles, a->seq_start, a->n_heads, a->n_kv_heads, a->head_dim,
-                 a->score_scale, a->softcap, a->window, a->status, a->sinks};
-    const int smem = QM * a->head_dim * 2 + 4 * KN * a->head_dim * 2 + QM * 128 + 1024;
+                 a->score_scale, a->softcap, a->window, a->status, a->sinks, a->chunk, a->rel_bias, a->rel_len, 0};
+    int smem = QM * a->head_dim * 2 + 4 * KN * a->head_dim * 2 + QM * 128 + 1024;
+    // a head's distance table lies beside the tiles where a multiprocessor holds as many blocks with it as without; else it
+    // is read through the cache (a block also has 1 KB that the system reserves and a little static shared memory)
+    const long long rel_bytes = a->rel_bias ? 4LL * a->rel_len : 0;
+    const int per_sm = 228 * 1024, beside = 1024 + 256;
+    const int room = per_sm / (per_sm / (smem + beside)) - beside;
+    if (a->rel_bias && smem + rel_bytes <= room) {
+        t.rel_in_smem = 1;
+        smem += (int)rel_bytes;
+    }
     dim3 grid(a->n_heads, a->n_tiles);
     switch (a->head_dim / 64) {
         case 1: return launch_tc<1>(grid, smem, (cudaStream_t)stream, map_q, map_kv, t);

@@ -115,6 +115,15 @@ __device__ __forceinline__ long long rdl_cache_offset(const int* __restrict__ ta
     return (((long long)page * n_kv_heads + kv_head) * page_size + r) * head_dim;
 }
 
+// The first key position a query at position p sees: the causal rule alone (0), a sliding window of `window` keys, or
+// chunks of `chunk` positions counted from the sequence's start, each seeing itself only (0 switches either off).
+__host__ __device__ __forceinline__ int rdl_first_key(int p, int window, int chunk) {
+    int lo = 0;
+    if (window > 0 && p - window + 1 > lo) lo = p - window + 1;
+    if (chunk > 0 && p - p % chunk > lo) lo = p - p % chunk;
+    return lo;
+}
+
 // Inside a row of a cache page the 16-byte chunks are stored swizzled by the row: chunk c of the row
 // at place `r` of its page lies at chunk c ^ (r & 7), for the chunks of the row's last incomplete
 // group of eight unchanged.  A whole [page_size][head_dim] block can then be copied to shared

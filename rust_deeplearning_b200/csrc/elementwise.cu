@@ -16,7 +16,8 @@
 // ---------------------------------------------------------------------------------------------
 __global__ void embed_rows_kernel(float* __restrict__ out, const void* __restrict__ table, int table_dtype,
                                   const int* __restrict__ ids, float scale, int hidden, int vocab,
-                                  int* __restrict__ status) {
+                                  int* __restrict__ status, const void* __restrict__ pos_table, int pos_dtype,
+                                  const int* __restrict__ tok_pos, int n_pos) {
     rdl_grid_wait();
     rdl_grid_launch_dependents();
     const int t = blockIdx.x;
@@ -29,17 +30,31 @@ __global__ void embed_rows_kernel(float* __restrict__ out, const void* __restric
         return;
     }
     const long long base = (long long)id * hidden;
-    for (int j = threadIdx.x; j < hidden; j += blockDim.x) o[j] = rdl_load(table, base + j, table_dtype) * scale;
+    const int p = pos_table ? tok_pos[t] : -1;          // a padding row (position -1) gets no position vector
+    if (p >= n_pos && pos_table) {
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x) o[j] = __int_as_float(0x7fc00000);
+        if (threadIdx.x == 0 && status) atomicExch(status, RDL_FAULT_POSITION);
+        return;
+    }
+    if (p < 0) {
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x) o[j] = rdl_load(table, base + j, table_dtype) * scale;
+    } else {
+        const long long pbase = (long long)p * hidden;
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x)
+            o[j] = rdl_load(table, base + j, table_dtype) * scale + rdl_load(pos_table, pbase + j, pos_dtype);
+    }
 }
 
 extern "C" int rdl_embed_rows(void* out_f32, const void* table, int table_dtype, const int* ids, float scale,
-                              int n_rows, int hidden, int vocab, int* status, void* stream) {
+                              int n_rows, int hidden, int vocab, int* status, const void* pos_table, int pos_dtype,
+                              const int* tok_pos, int n_pos, void* stream) {
     RDL_REQUIRE(rdl_valid_dtype(table_dtype), "embed_rows: bad table dtype %d", table_dtype);
     RDL_REQUIRE(n_rows >= 0 && hidden > 0 && vocab > 0, "embed_rows: bad sizes rows=%d hidden=%d vocab=%d", n_rows, hidden, vocab);
+    RDL_REQUIRE(!pos_table || (rdl_valid_dtype(pos_dtype) && tok_pos && n_pos > 0), "embed_rows: a position table comes with positions and its length");
     if (n_rows == 0) return 0;
     const int threads = hidden >= 1024 ? 256 : 128;
     RDL_CHECK_EX(rdl_launch(embed_rows_kernel, dim3(n_rows), dim3(threads), 0, (cudaStream_t)stream, (float*)out_f32, table,
-                            table_dtype, ids, scale, hidden, vocab, status), "embed_rows");
+                            table_dtype, ids, scale, hidden, vocab, status, pos_table, pos_dtype, tok_pos, n_pos), "embed_rows");
     return 0;
 }
 
@@ -283,10 +298,10 @@ extern "C" int rdl_norm_residual_norm(const void* x, int x_dtype, const int* row
 }
 
 // ---------------------------------------------------------------------------------------------
-// gated activation: out[t, i] = act(gu[t, i]) * gu[t, I + i]
+// gated activation: out[t, i] = gated(gu[t, i], gu[t, I + i]), act(g) * u or a form with a parameter
 // ---------------------------------------------------------------------------------------------
 __global__ void gated_activation_kernel(void* __restrict__ out, const void* __restrict__ gu, int dtype, int act,
-                                        long long n_rows, int inter) {
+                                        float param, long long n_rows, int inter) {
     const long long total = n_rows * inter;
     for (long long idx = blockIdx.x * (long long)blockDim.x + threadIdx.x; idx < total;
          idx += (long long)gridDim.x * blockDim.x) {
@@ -294,14 +309,13 @@ __global__ void gated_activation_kernel(void* __restrict__ out, const void* __re
         const int i = (int)(idx - t * inter);
         const float g = rdl_load(gu, t * 2 * inter + i, dtype);
         const float u = rdl_load(gu, t * 2 * inter + inter + i, dtype);
-        const float a = rdl_activation(g, act);
-        rdl_store(out, idx, dtype, a * u);
+        rdl_store(out, idx, dtype, rdl_gated(g, u, act, param));
     }
 }
 
 // bfloat16 rows whose width is a multiple of 8: eight values (16 bytes) of gate and of up per thread
 __global__ void gated_activation_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gu, int act,
-                                               long long n_rows, int inter) {
+                                               float param, long long n_rows, int inter) {
     const int chunks = inter >> 3;
     const long long total = n_rows * chunks;
     for (long long idx = blockIdx.x * (long long)blockDim.x + threadIdx.x; idx < total;
@@ -317,18 +331,16 @@ __global__ void gated_activation_bf16x8_kernel(__nv_bfloat16* __restrict__ out, 
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const float2 g = __bfloat1622float2(g2[i]), u = __bfloat1622float2(u2[i]);
-            const float a0 = rdl_activation(g.x, act);
-            const float a1 = rdl_activation(g.y, act);
-            r2[i] = __floats2bfloat162_rn(a0 * u.x, a1 * u.y);
+            r2[i] = __floats2bfloat162_rn(rdl_gated(g.x, u.x, act, param), rdl_gated(g.y, u.y, act, param));
         }
         *reinterpret_cast<uint4*>(out + t * inter + c * 8) = res;
     }
 }
 
 extern "C" int rdl_gated_activation(void* out, const void* gate_up, int dtype, int activation, int n_rows, int inter,
-                                    void* stream) {
+                                    float act_param, void* stream) {
     RDL_REQUIRE(rdl_valid_dtype(dtype), "gated_activation: bad dtype %d", dtype);
-    RDL_REQUIRE(rdl_activation_known(activation), "gated_activation: unknown activation %d", activation);
+    RDL_REQUIRE(rdl_gated_known(activation), "gated_activation: unknown activation %d", activation);
     RDL_REQUIRE(n_rows >= 0 && inter > 0, "gated_activation: bad sizes");
     if (n_rows == 0) return 0;
     const long long total = (long long)n_rows * inter;
@@ -336,13 +348,13 @@ extern "C" int rdl_gated_activation(void* out, const void* gate_up, int dtype, i
     if (dtype == RDL_BF16 && inter % 8 == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)gate_up & 15) == 0) {
         const long long blocks8 = (total / 8 + threads - 1) / threads;
         gated_activation_bf16x8_kernel<<<(unsigned)(blocks8 > rdl_sm_count() * 32 ? rdl_sm_count() * 32 : blocks8), threads, 0, (cudaStream_t)stream>>>(
-            (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, activation, n_rows, inter);
+            (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, activation, act_param, n_rows, inter);
         RDL_CHECK_LAUNCH("gated_activation");
         return 0;
     }
     const long long blocks = (total + threads - 1) / threads;
     gated_activation_kernel<<<(unsigned)(blocks > rdl_sm_count() * 16 ? rdl_sm_count() * 16 : blocks), threads, 0, (cudaStream_t)stream>>>(
-        out, gate_up, dtype, activation, n_rows, inter);
+        out, gate_up, dtype, activation, act_param, n_rows, inter);
     RDL_CHECK_LAUNCH("gated_activation");
     return 0;
 }

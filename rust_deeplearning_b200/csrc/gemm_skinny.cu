@@ -54,6 +54,7 @@ struct SkinnyArgs {
     int M, N, K;
     int out_dtype;              // RDL_F32 / RDL_BF16
     int activation;             // of the gated form
+    float act_param;            // the parameter of a gated form that has one
     float softcap;              // > 0: cap * tanh(v / cap)
     long long wait_cycles;      // clock cycles after which a wait is given up
     int test_extra_tx;          // tests only: bytes announced beyond what the block's first copy delivers
@@ -389,7 +390,7 @@ __global__ void __launch_bounds__(ST_THREADS, 2) gemm_stream_kernel(const __grid
                         if (GATED) { h1 += partial[w][0][slot + 8]; a1 += partial[w][IA][slot_a + 8]; }
                     }
                     float y = sc.y * (h0 + sc.x * a0);
-                    if (GATED) y = rdl_activation(y, a.activation) * (sc.y * (h1 + sc.x * a1));
+                    if (GATED) y = rdl_gated(y, sc.y * (h1 + sc.x * a1), a.activation, a.act_param);
                     if (a.softcap > 0.f) y = a.softcap * tanhf(y / a.softcap);
                     rdl_store(a.out, (long long)j * a.N + n, a.out_dtype, y);
                 }
@@ -406,7 +407,7 @@ __global__ void __launch_bounds__(ST_THREADS, 2) gemm_stream_kernel(const __grid
                     if (GATED) v1 += partial[w][i][slot + 8];
                 }
                 float y = v0;
-                if (GATED) y = rdl_activation(v0, a.activation) * v1;
+                if (GATED) y = rdl_gated(v0, v1, a.activation, a.act_param);
                 else if (a.activation >= 16) y = rdl_unary(v0, a.activation);     // an element-wise activation of the plain form
                 if (a.softcap > 0.f) y = a.softcap * tanhf(y / a.softcap);
                 rdl_store(a.out, (long long)m * a.N + n, a.out_dtype, y);
@@ -450,16 +451,16 @@ void launch_stream(const SkinnyArgs& a, int* status, cudaStream_t st) {
 }  // namespace
 
 extern "C" int rdl_gemm_skinny(void* out, int out_dtype, const void* x, const void* w, int m, int n, int k,
-                               int gated, int activation, float softcap, int* status, void* stream) {
+                               int gated, int activation, float softcap, int* status, float act_param, void* stream) {
     RDL_REQUIRE(out && x && w, "gemm_skinny: missing operand");
     RDL_REQUIRE(rdl_valid_dtype(out_dtype), "gemm_skinny: bad output dtype %d", out_dtype);
     RDL_REQUIRE(m >= 0 && m <= 16, "gemm_skinny: %d rows, at most 16 are supported", m);
     RDL_REQUIRE(n > 0 && k > 0 && k % 8 == 0, "gemm_skinny: n=%d, k=%d; k must be a multiple of 8", n, k);
     RDL_REQUIRE((uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0, "gemm_skinny: operands must start on 16-byte boundaries");
-    RDL_REQUIRE(!gated || rdl_activation_known(activation), "gemm_skinny: unknown activation %d", activation);
+    RDL_REQUIRE(!gated || rdl_gated_known(activation), "gemm_skinny: unknown activation %d", activation);
     RDL_REQUIRE(softcap >= 0.f, "gemm_skinny: soft-cap must not be negative");
     if (m == 0) return 0;
-    SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out, m, n, k, out_dtype, activation, softcap,
+    SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out, m, n, k, out_dtype, activation, act_param, softcap,
                  rdl_wait_cycles_for(RDL_FAULT_GEMM_STREAM), rdl_test_extra_tx_for(RDL_FAULT_GEMM_STREAM), DeferredNormArgs{}};
     cudaStream_t st = (cudaStream_t)stream;
     g_launch_error = cudaSuccess;
@@ -476,14 +477,14 @@ extern "C" int rdl_gemm_skinny(void* out, int out_dtype, const void* x, const vo
 
 extern "C" int rdl_gemm_skinny_norm(void* out, int out_dtype, const void* x, const void* w, int m, int n, int k,
                                     int gated, int activation, float softcap, const DeferredNormArgs* norm, int* status,
-                                    void* stream) {
+                                    float act_param, void* stream) {
     RDL_REQUIRE(x && w && norm, "gemm_skinny_norm: missing operand");
     RDL_REQUIRE(m >= 0 && m <= 8, "gemm_skinny_norm: %d rows, at most 8 are supported", m);
     RDL_REQUIRE(n > 0 && k > 0 && k % 8 == 0, "gemm_skinny_norm: n=%d, k=%d; k must be a multiple of 8", n, k);
     RDL_REQUIRE((uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0, "gemm_skinny_norm: operands must start on 16-byte boundaries");
     RDL_REQUIRE(norm->sums && (uintptr_t)norm->sums % 16 == 0, "gemm_skinny_norm: the partial sums must lie on a 16-byte boundary");
     if (m == 0) return 0;
-    SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out, m, n, k, out_dtype, activation, softcap,
+    SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out, m, n, k, out_dtype, activation, act_param, softcap,
                  rdl_wait_cycles_for(RDL_FAULT_GEMM_STREAM), rdl_test_extra_tx_for(RDL_FAULT_GEMM_STREAM), *norm};
     cudaStream_t st = (cudaStream_t)stream;
     g_launch_error = cudaSuccess;
@@ -494,7 +495,7 @@ extern "C" int rdl_gemm_skinny_norm(void* out, int out_dtype, const void* x, con
         launch_stream<1, false, 1>(a, status, st);
     } else if (norm->mode == RDL_NORM_DEFERRED) {
         RDL_REQUIRE(out && rdl_valid_dtype(out_dtype), "gemm_skinny_norm: missing output or bad output dtype %d", out_dtype);
-        RDL_REQUIRE(!gated || rdl_activation_known(activation), "gemm_skinny_norm: unknown activation %d", activation);
+        RDL_REQUIRE(!gated || rdl_gated_known(activation), "gemm_skinny_norm: unknown activation %d", activation);
         RDL_REQUIRE(softcap >= 0.f, "gemm_skinny_norm: soft-cap must not be negative");
         RDL_REQUIRE(norm->n_sums > 0 && norm->n_out >= 0 && norm->n_out <= 8, "gemm_skinny_norm: %d units of sums, %d output rows", norm->n_sums, norm->n_out);
         const bool side = norm->residual_out || norm->scaled_next;

@@ -599,13 +599,13 @@ int launch_pair(const CUtensorMap& mx, const CUtensorMap& mw, const TcArgs& a, c
 }  // namespace
 
 extern "C" int rdl_gemm_tc(void* out, int out_dtype, const void* x, const void* w, int m, int n, int k,
-                           int gated, int activation, float softcap, int* status, void* stream) {
+                           int gated, int activation, float softcap, int* status, float act_param, void* stream) {
     RDL_REQUIRE(out && x && w, "gemm_tc: missing operand");
     RDL_REQUIRE(rdl_valid_dtype(out_dtype), "gemm_tc: bad output dtype %d", out_dtype);
     RDL_REQUIRE(m >= 0 && n > 0 && k > 0 && k % 8 == 0, "gemm_tc: m=%d n=%d k=%d; k must be a multiple of 8", m, n, k);
     RDL_REQUIRE((uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0,
                 "gemm_tc: operands must start on 16-byte boundaries");
-    RDL_REQUIRE(!gated || rdl_activation_known(activation), "gemm_tc: unknown activation %d", activation);
+    RDL_REQUIRE(!gated || rdl_gated_known(activation), "gemm_tc: unknown activation %d", activation);
     RDL_REQUIRE(softcap >= 0.f, "gemm_tc: soft-cap must not be negative");
     if (m == 0) return 0;
     // Pairs of multiprocessors on 256 x 256 tiles where a tile's products are many (the gated form, or a long
@@ -632,7 +632,7 @@ extern "C" int rdl_gemm_tc(void* out, int out_dtype, const void* x, const void* 
         }
         mw = it->second;
     }
-    TcArgs a{out, m, n, k, out_dtype, activation, softcap, status, nullptr, 0, 0.f};
+    TcArgs a{out, m, n, k, out_dtype, activation, softcap, status, nullptr, 0, act_param};
     cudaStream_t st = (cudaStream_t)stream;
     if (pair) {
         // a second accumulator (the products of a tile run while the tile before it is stored) where a pair

@@ -4,6 +4,9 @@
 //   z = W_r x,  s = softmax(z) over all experts (identity experts included), or s = sigmoid(z) expert by expert,
 //   choice = s + correction;  the `top` largest choices are taken (ties: the lower index),
 //   their weights are s itself (not renormalised).
+//   Groups (optional): the experts form equal groups of neighbours; only those of the groups with the largest scores (the
+//   sum of a group's two largest choices) can be chosen.  Normalised (optional): the weights are divided by their sum.
+//   Extra rows (optional) of W_r beyond the experts only form logits: a number per token for whoever reads them.
 //   A third scoring: z = W_r x + b, the `top` largest z are taken and their weights are the softmax over those z alone.
 // An expert e < n_real is a gated feed-forward, y = W_down act(W_gate x, W_up x); an expert e >= n_real is
 // an identity expert whose output is x.  The row's result is sum_k weight_k y_k in the order of the choice.
@@ -135,19 +138,20 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_logits_kernel(const T* _
 constexpr int TOPK_WARPS = 4;
 
 __global__ void __launch_bounds__(TOPK_WARPS * 32) moe_topk_kernel(const float* __restrict__ z, const float* __restrict__ bias,
-                                                                   const float* __restrict__ correction, int n_rows,
-                                                                   int n_experts, int top, int scoring, int* __restrict__ sel,
-                                                                   float* __restrict__ sel_w) {
-    extern __shared__ float zs_all[];          // per warp: [n_experts] scores, [n_experts] choices, [top] chosen scores
+                                                                   const float* __restrict__ correction, int n_rows, int z_stride,
+                                                                   int n_experts, int top, int scoring, int n_groups, int keep,
+                                                                   float norm_eps, int* __restrict__ sel, float* __restrict__ sel_w) {
+    extern __shared__ float zs_all[];          // per warp: [n_experts] scores, [n_experts] choices, [top] chosen scores, [n_groups] groups
     rdl_grid_wait();
     rdl_grid_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * TOPK_WARPS + warp;
     if (t >= n_rows) return;
-    float* zs = zs_all + (size_t)warp * (2 * n_experts + top);
+    float* zs = zs_all + (size_t)warp * (2 * n_experts + top + n_groups);
     float* choice = zs + n_experts;
     float* picked = choice + n_experts;
-    const float* zr = z + (long long)t * n_experts;
+    float* group = picked + top;
+    const float* zr = z + (long long)t * z_stride;
     float m = -INFINITY;
     float sum = 1.f;
     auto logit = [&](int e) { return bias ? zr[e] + bias[e] : zr[e]; };
@@ -173,6 +177,40 @@ __global__ void __launch_bounds__(TOPK_WARPS * 32) moe_topk_kernel(const float* 
         choice[e] = s + (correction ? correction[e] : 0.f);
     }
     __syncwarp();
+    if (n_groups > 0) {
+        // groups of neighbours: a group's score is the sum of its two largest choices; experts of groups outside the `keep`
+        // best (ties: the lower index) cannot be chosen
+        const int size = n_experts / n_groups;
+        for (int gi = lane; gi < n_groups; gi += 32) {
+            float first = -INFINITY, second = -INFINITY;
+            for (int i = 0; i < size; ++i) {
+                const float c = choice[gi * size + i];
+                if (c > first) { second = first; first = c; }
+                else if (c > second) second = c;
+            }
+            group[gi] = size > 1 ? first + second : first;
+        }
+        __syncwarp();
+        for (int k = 0; k < n_groups - keep; ++k) {          // rule out the smallest (ties: the higher index goes first)
+            float worst = INFINITY;
+            int worst_g = -1;
+            for (int gi = lane; gi < n_groups; gi += 32) {
+                const float c = group[gi];
+                if (c <= worst) { worst = c; worst_g = gi; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ow = __shfl_xor_sync(0xffffffffu, worst, o);
+                const int og = __shfl_xor_sync(0xffffffffu, worst_g, o);
+                if (ow < worst || (ow == worst && og > worst_g)) { worst = ow; worst_g = og; }
+            }
+            if (worst_g < 0) break;                           // only if every remaining score is NaN
+            for (int i = lane; i < size; i += 32) choice[worst_g * size + i] = -INFINITY;
+            __syncwarp();
+            if (lane == 0) group[worst_g] = INFINITY;         // ruled out: never the smallest again
+            __syncwarp();
+        }
+    }
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int best_e = 0x7fffffff;
@@ -189,7 +227,7 @@ __global__ void __launch_bounds__(TOPK_WARPS * 32) moe_topk_kernel(const float* 
         if (best_e == 0x7fffffff) best_e = 0;              // only if every remaining choice is NaN or -inf
         if (lane == 0) {
             sel[(long long)t * top + k] = best_e;
-            if (scoring == RDL_ROUTE_SOFTMAX_CHOSEN) picked[k] = zs[best_e];
+            if (scoring == RDL_ROUTE_SOFTMAX_CHOSEN || norm_eps > 0.f) picked[k] = zs[best_e];
             else sel_w[(long long)t * top + k] = zs[best_e];
             choice[best_e] = -INFINITY;
         }
@@ -201,6 +239,11 @@ __global__ void __launch_bounds__(TOPK_WARPS * 32) moe_topk_kernel(const float* 
         float total = 0.f;
         for (int k = 0; k < top; ++k) { picked[k] = expf(picked[k] - top_logit); total += picked[k]; }
         for (int k = 0; k < top; ++k) sel_w[(long long)t * top + k] = picked[k] / total;
+    } else if (norm_eps > 0.f && lane == 0) {
+        // the weights: the chosen scores divided by their sum, added up in the order of the choice
+        float total = 0.f;
+        for (int k = 0; k < top; ++k) total += picked[k];
+        for (int k = 0; k < top; ++k) sel_w[(long long)t * top + k] = picked[k] / (total + norm_eps);
     }
 }
 
@@ -453,11 +496,15 @@ __global__ void moe_combine_kernel(__nv_bfloat16* __restrict__ out, const __nv_b
 }  // namespace
 
 extern "C" int rdl_moe_route(const void* x, int dtype, const float* w_router, const float* bias, const float* correction, int n_rows,
-                             int n_experts, int width, int top, int scoring, int* sel, float* sel_w, float* logits, void* stream) {
+                             int n_experts, int width, int top, int scoring, int* sel, float* sel_w, float* logits, int extra, int n_groups,
+                             int keep, float norm_eps, void* stream) {
     RDL_REQUIRE(rdl_valid_dtype(dtype), "moe_route: bad dtype %d", dtype);
     RDL_REQUIRE(x && w_router && sel && sel_w && logits && n_experts > 0 && width > 0, "moe_route: bad arguments");
     RDL_REQUIRE(top >= 1 && top <= n_experts, "moe_route: %d of %d experts cannot be chosen", top, n_experts);
     RDL_REQUIRE(scoring == RDL_ROUTE_SOFTMAX || scoring == RDL_ROUTE_SIGMOID || scoring == RDL_ROUTE_SOFTMAX_CHOSEN, "moe_route: unknown scoring %d", scoring);
+    RDL_REQUIRE(extra >= 0 && norm_eps >= 0.f && !(norm_eps > 0.f && scoring == RDL_ROUTE_SOFTMAX_CHOSEN), "moe_route: bad extra rows or normalisation");
+    RDL_REQUIRE(n_groups >= 0 && (n_groups == 0 || (n_experts % n_groups == 0 && keep >= 1 && keep <= n_groups && top <= keep * (n_experts / n_groups))),
+                "moe_route: %d experts in %d groups of which %d are kept cannot give %d choices", n_experts, n_groups, keep, top);
     RDL_REQUIRE(n_experts <= 1024, "moe_route: %d experts exceed the 1,024 the router kernels hold", n_experts);
     if (n_rows == 0) return 0;
     cudaStream_t st = (cudaStream_t)stream;
@@ -466,20 +513,21 @@ extern "C" int rdl_moe_route(const void* x, int dtype, const float* w_router, co
     // row count, always takes the first)
     const bool few = n_rows <= 64 || dtype == RDL_F32;
     const dim3 block(ROUTE_WARPS * 32);
-    const dim3 grid = few ? dim3((n_rows + ROUTE_FEW_ROWS - 1) / ROUTE_FEW_ROWS, n_experts)
-                          : dim3((n_rows + ROUTE_MANY_ROWS - 1) / ROUTE_MANY_ROWS, (n_experts + ROUTE_WARPS - 1) / ROUTE_WARPS);
+    const int n_logits = n_experts + extra;
+    const dim3 grid = few ? dim3((n_rows + ROUTE_FEW_ROWS - 1) / ROUTE_FEW_ROWS, n_logits)
+                          : dim3((n_rows + ROUTE_MANY_ROWS - 1) / ROUTE_MANY_ROWS, (n_logits + ROUTE_WARPS - 1) / ROUTE_WARPS);
     if (dtype == RDL_BF16) {
         const __nv_bfloat16* xp = (const __nv_bfloat16*)x;
-        if (few) RDL_CHECK_EX(rdl_launch(moe_logits_kernel<__nv_bfloat16, ROUTE_FEW_ROWS, true>, grid, block, 0, st, xp, w_router, n_rows, n_experts, width, logits), "moe_route");
-        else RDL_CHECK_EX(rdl_launch(moe_logits_kernel<__nv_bfloat16, ROUTE_MANY_ROWS, false>, grid, block, 0, st, xp, w_router, n_rows, n_experts, width, logits), "moe_route");
+        if (few) RDL_CHECK_EX(rdl_launch(moe_logits_kernel<__nv_bfloat16, ROUTE_FEW_ROWS, true>, grid, block, 0, st, xp, w_router, n_rows, n_logits, width, logits), "moe_route");
+        else RDL_CHECK_EX(rdl_launch(moe_logits_kernel<__nv_bfloat16, ROUTE_MANY_ROWS, false>, grid, block, 0, st, xp, w_router, n_rows, n_logits, width, logits), "moe_route");
     } else {
         const float* xp = (const float*)x;
-        if (few) RDL_CHECK_EX(rdl_launch(moe_logits_kernel<float, ROUTE_FEW_ROWS, true>, grid, block, 0, st, xp, w_router, n_rows, n_experts, width, logits), "moe_route");
-        else RDL_CHECK_EX(rdl_launch(moe_logits_kernel<float, ROUTE_MANY_ROWS, false>, grid, block, 0, st, xp, w_router, n_rows, n_experts, width, logits), "moe_route");
+        if (few) RDL_CHECK_EX(rdl_launch(moe_logits_kernel<float, ROUTE_FEW_ROWS, true>, grid, block, 0, st, xp, w_router, n_rows, n_logits, width, logits), "moe_route");
+        else RDL_CHECK_EX(rdl_launch(moe_logits_kernel<float, ROUTE_MANY_ROWS, false>, grid, block, 0, st, xp, w_router, n_rows, n_logits, width, logits), "moe_route");
     }
-    const size_t smem = (size_t)TOPK_WARPS * (2 * n_experts + top) * sizeof(float);
+    const size_t smem = (size_t)TOPK_WARPS * (2 * n_experts + top + n_groups) * sizeof(float);
     RDL_CHECK_EX(rdl_launch(moe_topk_kernel, dim3((n_rows + TOPK_WARPS - 1) / TOPK_WARPS), dim3(TOPK_WARPS * 32), smem, st, (const float*)logits,
-                            bias, correction, n_rows, n_experts, top, scoring, sel, sel_w), "moe_route");
+                            bias, correction, n_rows, n_logits, n_experts, top, scoring, n_groups, keep, norm_eps, sel, sel_w), "moe_route");
     return 0;
 }
 

@@ -1,0 +1,286 @@
+// Everything between the q/k/v product and attention for designs with a short convolution on the projections, in one pass:
+//   u   = row + bias                                        (the projection; the bias optional)
+//   c_t = sum_j conv[:, j] u_(t - (taps - 1) + j)           per channel along the sequence, zeros before its start (optional)
+//   q   = c / sqrt(sum over ALL query channels of c^2 / q_count + eps) * wq,   k likewise with k_count and wk   (optional)
+//   v   = (1 - lambda) c + lambda first                     (another layer's values of the same token; optional)
+// and the cache write of k and v.  All in float; every value is rounded once, on its way into the packed rows the attention
+// kernels read and into the cache.  q_count and k_count are the projections' sizes without any zero padding of their heads.
+//
+// A sequence's last taps - 1 values of u are state per slot (float [slots][taps - 1][channels]): a step's first tokens read
+// what the step before left, and the block of a sequence's first tokens leaves the last ones.
+//
+// A block takes QP_GROUP consecutive tokens of one sequence (a group starts at a multiple of QP_GROUP within the step's rows of
+// the sequence; the blocks of the other tokens end at once), NT of them at a time; a thread owns the same channels for all
+// of them, so a row that several outputs need is loaded once a group of NT, and the state is read and written by the thread that
+// owns the channel: the first group reads all the state a step's tokens need (QP_GROUP > taps - 1) before it writes.
+// The sums of squares are formed thread by thread, then across each warp, then over the warps in rising order: an order that
+// depends on the number of channels alone, never on the step's rows, on the cut or on NT.
+#include "api.h"
+#include "common.cuh"
+#include "launch.cuh"
+
+namespace {
+
+constexpr int QP_GROUP = 8, QP_MAX_TAPS = 8;
+
+template <typename T> struct Piece;
+template <> struct Piece<__nv_bfloat16> {
+    static constexpr int N = 8;
+    static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&f)[8]) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(p);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { const float2 v = __bfloat1622float2(h[i]); f[2 * i] = v.x; f[2 * i + 1] = v.y; }
+    }
+    static __device__ __forceinline__ uint4 pack(const float (&f)[8]) {
+        uint4 raw;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+        return raw;
+    }
+};
+template <> struct Piece<float> {
+    static constexpr int N = 4;
+    static __device__ __forceinline__ void load(const float* p, float (&f)[4]) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+    }
+    static __device__ __forceinline__ uint4 pack(const float (&f)[4]) {
+        return make_uint4(__float_as_uint(f[0]), __float_as_uint(f[1]), __float_as_uint(f[2]), __float_as_uint(f[3]));
+    }
+};
+
+// VEC: pieces of 16 bytes (head_dim a whole number of them), else single values.  CPT: pieces a thread owns.  NT: tokens at a
+// time.  TAPS: the most taps this instance takes.
+template <typename T, bool VEC, int CPT, int NT, int TAPS>
+__global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepareArgs a) {
+    constexpr int N = VEC ? Piece<T>::N : 1;
+    __shared__ float part[2 * NT][32];
+    const int t0 = blockIdx.x;
+    const int pos0 = a.tok_pos[t0];
+    if (pos0 < 0) return;                                   // a padding row of a fixed-size batch
+    const int seq = a.tok_seq[t0], row0 = a.seq_start[seq], r0 = t0 - row0;
+    if (r0 % QP_GROUP) return;                              // the block of the group's first token takes it
+    const int n = a.seq_start[seq + 1] - row0, past = pos0 - r0;
+    const int C = a.n_channels, D = a.head_dim, qw = a.n_heads * D, kw = a.n_kv_heads * D;
+    const int taps = a.conv ? a.taps : 1, keep = taps - 1;
+    const T* rows = (const T*)a.rows + (long long)row0 * a.row_stride;      // the sequence's rows of this step
+    T* out = (T*)a.out + (long long)row0 * a.out_stride;
+    const T* first = a.v_first ? (const T*)a.v_first + (long long)row0 * a.v_first_stride : nullptr;
+    const T* conv = (const T*)a.conv;
+    float* st = keep > 0 ? a.state + (long long)a.slots[seq] * keep * C : nullptr;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    auto load = [](const T* p, float (&f)[N]) {
+        if constexpr (VEC) Piece<T>::load(p, f);
+        else f[0] = to_float(*p);
+    };
+    auto floats = [](const float* p, float (&f)[N]) {
+        if constexpr (VEC) {
+#pragma unroll
+            for (int e = 0; e < N; e += 4) {
+                const float4 v = *reinterpret_cast<const float4*>(p + e);
+                f[e] = v.x; f[e + 1] = v.y; f[e + 2] = v.z; f[e + 3] = v.w;
+            }
+        } else {
+            f[0] = *p;
+        }
+    };
+    auto store = [](T* p, const float (&f)[N]) {
+        if constexpr (VEC) *reinterpret_cast<uint4*>(p) = Piece<T>::pack(f);
+        else *p = from_float<T>(f[0]);
+    };
+    // u of the step's row `src` (below zero: from the state, or zeros before the sequence's start)
+    auto projected = [&](int src, int c, const float (&bias)[N], float (&u)[N]) {
+        if (src >= 0) {
+            load(rows + (long long)src * a.row_stride + c, u);
+#pragma unroll
+            for (int e = 0; e < N; ++e) u[e] += bias[e];
+        } else if (past + src >= 0) {
+            floats(st + (long long)(keep + src) * C + c, u);
+        } else {
+#pragma unroll
+            for (int e = 0; e < N; ++e) u[e] = 0.f;
+        }
+    };
+    rdl_grid_wait();
+    rdl_grid_launch_dependents();
+    const int end = min(r0 + QP_GROUP, n);
+    for (int rb = r0; rb < end; rb += NT) {
+        float acc[NT][CPT][N];
+        float sums[2 * NT];
+#pragma unroll
+        for (int i = 0; i < 2 * NT; ++i) sums[i] = 0.f;
+#pragma unroll
+        for (int it = 0; it < CPT; ++it) {
+            const int c = (threadIdx.x + it * blockDim.x) * N;
+#pragma unroll
+            for (int i = 0; i < NT; ++i)
+#pragma unroll
+                for (int e = 0; e < N; ++e) acc[i][it][e] = 0.f;
+            if (c < C) {
+                float bias[N], w[TAPS][N];
+#pragma unroll
+                for (int e = 0; e < N; ++e) bias[e] = 0.f;
+                if (a.bias) floats(a.bias + c, bias);
+                // w[k]: the weight of the value k tokens back
+#pragma unroll
+                for (int k = 0; k < TAPS; ++k) {
+                    if (k <= keep && conv) load(conv + (long long)(keep - k) * C + c, w[k]);
+                    else
+#pragma unroll
+                        for (int e = 0; e < N; ++e) w[k][e] = k == 0 ? 1.f : 0.f;
+                }
+#pragma unroll
+                for (int rr = -(TAPS - 1); rr < NT; ++rr) {
+                    const int src = rb + rr;
+                    if (rr < -keep || src >= n) continue;
+                    float u[N];
+                    projected(src, c, bias, u);
+#pragma unroll
+                    for (int i = 0; i < NT; ++i) {
+                        const int k = i - rr;               // row rr counts k tokens back for token i
+                        if (k >= 0 && k < TAPS)
+#pragma unroll
+                            for (int e = 0; e < N; ++e) acc[i][it][e] = fmaf(w[k][e], u[e], acc[i][it][e]);
+                    }
+                }
+                if (c < qw + kw) {
+#pragma unroll
+                    for (int i = 0; i < NT; ++i) {
+                        float s = 0.f;
+#pragma unroll
+                        for (int e = 0; e < N; ++e) s = fmaf(acc[i][it][e], acc[i][it][e], s);
+                        sums[2 * i] += c < qw ? s : 0.f;
+                        sums[2 * i + 1] += c < qw ? 0.f : s;
+                    }
+                }
+            }
+        }
+        float inv[2 * NT];
+        if (a.wq) {
+            __syncthreads();                                // the sums of the tokens before are no longer read
+#pragma unroll
+            for (int i = 0; i < 2 * NT; ++i) {
+                const float s = warp_sum(sums[i]);
+                if (lane == 0) part[i][warp] = s;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int i = 0; i < 2 * NT; ++i) {
+                float s = 0.f;
+                for (int wdx = 0; wdx < n_warps; ++wdx) s += part[i][wdx];
+                inv[i] = 1.0f / sqrtf(s / ((i & 1) ? a.k_count : a.q_count) + a.eps);
+            }
+        }
+#pragma unroll
+        for (int it = 0; it < CPT; ++it) {
+            const int c = (threadIdx.x + it * blockDim.x) * N;
+            if (c >= C) continue;
+            const bool is_q = c < qw, is_k = !is_q && c < qw + kw;
+            float wn[N];
+            if (a.wq && (is_q || is_k)) floats(is_q ? a.wq + c : a.wk + (c - qw), wn);
+            const int head = is_q ? 0 : (is_k ? c - qw : c - qw - kw) / D;
+            const int d = is_q ? 0 : (is_k ? c - qw : c - qw - kw) - head * D;
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                const int r = rb + i;
+                if (r >= end) continue;
+                float (&v)[N] = acc[i][it];
+                if (is_q || is_k) {
+                    if (a.wq) {
+                        const float s = is_q ? inv[2 * i] : inv[2 * i + 1];
+#pragma unroll
+                        for (int e = 0; e < N; ++e) v[e] = v[e] * s * wn[e];
+                    }
+                } else if (first) {
+                    float f[N];
+                    load(first + (long long)r * a.v_first_stride + (c - qw - kw), f);
+#pragma unroll
+                    for (int e = 0; e < N; ++e) v[e] = (1.0f - a.v_lambda) * v[e] + a.v_lambda * f[e];
+                }
+                store(out + (long long)r * a.out_stride + c, v);
+                if (is_q || !a.do_write) continue;
+                const int p = past + r;
+                // In a ring a later token of this step may land on the same row: only the last writer writes.
+                if ((long long)p + (long long)a.ring_pages * a.page_size < (long long)a.seq_end[seq]) continue;
+                T* dst = (T*)(is_k ? a.k_cache : a.v_cache) +
+                         rdl_cache_offset(a.tables + (long long)seq * a.table_width, p, a.page_size, a.ring_pages, a.n_kv_heads, head, D);
+                const int pr = p % a.page_size;             // chunks of a cache row are stored swizzled by its place in the page
+                store(dst + (VEC ? rdl_swizzled_chunk(pr, d / N, D / N) * N : rdl_cache_col<T>(pr, d, D)), v);
+            }
+        }
+    }
+    if (r0 == 0 && keep > 0) {
+        // the sequence's last taps - 1 values of u, in rising order: an entry is read before it is written (row j takes an
+        // older entry j + n > j, or a row of the step)
+#pragma unroll
+        for (int it = 0; it < CPT; ++it) {
+            const int c = (threadIdx.x + it * blockDim.x) * N;
+            if (c >= C) continue;
+            float bias[N];
+#pragma unroll
+            for (int e = 0; e < N; ++e) bias[e] = 0.f;
+            if (a.bias) floats(a.bias + c, bias);
+            for (int j = 0; j < keep; ++j) {
+                float u[N];
+                projected(n - keep + j, c, bias, u);
+#pragma unroll
+                for (int e = 0; e < N; ++e) st[(long long)j * C + c + e] = u[e];
+            }
+        }
+    }
+}
+
+template <typename T, bool VEC, int CPT, int NT>
+cudaError_t launch_prepare(const QkvPrepareArgs& a, int threads, cudaStream_t st) {
+    if (a.conv && a.taps > 4) return rdl_launch(qkv_prepare_kernel<T, VEC, CPT, NT, QP_MAX_TAPS>, dim3(a.n_tokens), dim3(threads), 0, st, a);
+    return rdl_launch(qkv_prepare_kernel<T, VEC, CPT, NT, 4>, dim3(a.n_tokens), dim3(threads), 0, st, a);
+}
+
+// steps of single tokens take tokens one by one; prompts several at a time where a thread's registers hold them
+template <typename T>
+cudaError_t launch_prepare_for(const QkvPrepareArgs& a, bool vec, int pieces, cudaStream_t st) {
+    const bool single = a.n_tokens <= a.n_seqs;
+    auto threads_for = [&](int cpt) { const int t = ((pieces + cpt - 1) / cpt + 31) / 32 * 32; return t < 64 ? 64 : t; };
+    if (vec) {
+        if (pieces <= 512) return single ? launch_prepare<T, true, 1, 1>(a, threads_for(1), st) : launch_prepare<T, true, 1, 4>(a, threads_for(1), st);
+        if (pieces <= 1024) return single ? launch_prepare<T, true, 2, 1>(a, threads_for(2), st) : launch_prepare<T, true, 2, 2>(a, threads_for(2), st);
+        return launch_prepare<T, true, 4, 1>(a, threads_for(4), st);
+    }
+    if (pieces <= 1024) return launch_prepare<T, false, 1, 1>(a, threads_for(1), st);
+    if (pieces <= 4096) return launch_prepare<T, false, 4, 1>(a, threads_for(4), st);
+    return launch_prepare<T, false, 16, 1>(a, threads_for(16), st);
+}
+
+}  // namespace
+
+extern "C" int rdl_qkv_prepare(const QkvPrepareArgs* p, void* stream) {
+    QkvPrepareArgs a = *p;
+    RDL_REQUIRE(rdl_valid_dtype(a.dtype), "qkv_prepare: bad dtype %d", a.dtype);
+    RDL_REQUIRE(a.n_tokens >= 0 && a.n_seqs >= 0 && a.n_heads > 0 && a.n_kv_heads > 0 && a.head_dim > 0,
+                "qkv_prepare: bad sizes tokens=%d heads=%d kv_heads=%d head_dim=%d", a.n_tokens, a.n_heads, a.n_kv_heads, a.head_dim);
+    a.n_channels = (a.n_heads + 2 * a.n_kv_heads) * a.head_dim;
+    RDL_REQUIRE(a.rows && a.out && a.rows != a.out && a.row_stride >= a.n_channels && a.out_stride >= a.n_channels,
+                "qkv_prepare: rows in and out must be different buffers at least as wide as the heads");
+    RDL_REQUIRE(a.tok_seq && a.tok_pos && a.seq_start && a.slots && a.seq_end, "qkv_prepare: missing batch description");
+    RDL_REQUIRE(!a.conv || (a.taps >= 1 && a.taps <= QP_MAX_TAPS), "qkv_prepare: %d taps, the kernel takes 1 to %d", a.taps, QP_MAX_TAPS);
+    RDL_REQUIRE(!a.conv || a.taps == 1 || a.state, "qkv_prepare: more than one tap needs the slots' state");
+    RDL_REQUIRE((a.wq == nullptr) == (a.wk == nullptr) && (!a.wq || (a.eps > 0.f && a.q_count > 0.f && a.k_count > 0.f)),
+                "qkv_prepare: the norms need both weights, eps > 0 and the projections' true sizes");
+    RDL_REQUIRE(!a.v_first || a.v_first_stride >= (long long)a.n_kv_heads * a.head_dim, "qkv_prepare: the first values' rows are narrower than the heads");
+    RDL_REQUIRE(!a.do_write || (a.k_cache && a.v_cache && a.tables && a.page_size > 0 && a.ring_pages > 0 && a.ring_pages <= a.table_width),
+                "qkv_prepare: cache write needs storage and page tables");
+    if (a.n_tokens == 0) return 0;
+    const int per = a.dtype == RDL_BF16 ? 8 : 4;
+    const bool vec = a.head_dim % per == 0 && a.row_stride % per == 0 && a.out_stride % per == 0 && a.v_first_stride % per == 0 &&
+                     a.n_channels / per <= 2048 &&
+                     (((uintptr_t)a.rows | (uintptr_t)a.out | (uintptr_t)a.bias | (uintptr_t)a.conv | (uintptr_t)a.state | (uintptr_t)a.wq |
+                       (uintptr_t)a.wk | (uintptr_t)a.v_first | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache) & 15) == 0;
+    const int pieces = vec ? a.n_channels / per : a.n_channels;
+    RDL_REQUIRE(pieces <= 16384, "qkv_prepare: %d channels exceed the 16,384 the kernel holds", a.n_channels);
+    cudaStream_t st = (cudaStream_t)stream;
+    cudaError_t e = a.dtype == RDL_BF16 ? launch_prepare_for<__nv_bfloat16>(a, vec, pieces, st) : launch_prepare_for<float>(a, vec, pieces, st);
+    RDL_CHECK_EX(e, "qkv_prepare");
+    return 0;
+}

@@ -84,6 +84,7 @@ class StepBatch:
     # run -> the cache write it has put off until the runs that read its keys and values are through (a ring
     # group's rows of earlier steps are still needed by this step's readers); the model calls them
     deferred_writes: Dict[int, object] = field(default_factory=dict)
+    carried: Dict[str, object] = field(default_factory=dict)         # what one layer leaves of this step's rows for later ones, by name
     cache_owner_of: Dict[int, int] = field(default_factory=dict)     # run -> run whose keys and values it reads
     shared_runs: frozenset = frozenset()                             # runs whose keys and values a later run reads
     status: Optional[torch.Tensor] = None                            # int32 flag kernels set when they give up a wait

@@ -23,7 +23,7 @@ from concurrent.futures import ThreadPoolExecutor
 _PKG = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CSRC = os.path.join(_PKG, "csrc")
 LIB_NAME = "librdl_b200_kernels.so"
-ABI_VERSION = 19
+ABI_VERSION = 20
 
 # fast math is never enabled: the 32-bit path relies on exact tanhf/expf/sqrtf and plain FMA
 NVCC_FLAGS = ["-std=c++17", "-O3", "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo",
@@ -173,6 +173,7 @@ class AttentionArgs(ctypes.Structure):
         ("counter_bytes", ctypes.c_longlong), ("status", ctypes.c_void_p),
         ("rope_cos", ctypes.c_void_p), ("rope_sin", ctypes.c_void_p), ("rotary_dim", ctypes.c_int), ("new_rows", ctypes.c_int),
         ("sinks", ctypes.c_void_p), ("sigmoid_bias", ctypes.c_void_p),
+        ("chunk", ctypes.c_int), ("rel_bias", ctypes.c_void_p), ("rel_len", ctypes.c_int),
         ("wait_cycles", ctypes.c_longlong), ("test_extra_tx", ctypes.c_int),     # filled in by the launcher
     ]
 
@@ -180,6 +181,7 @@ class AttentionArgs(ctypes.Structure):
 # What a kernel leaves in a step's status word when it gives up (`csrc/api.h`, RDL_FAULT_*).
 FAULTS = {
     1: "embed_rows: a token id outside the vocabulary (its row is NaN)",
+    2: "embed_rows: a position beyond the position table (its row is NaN)",
     3: "attention_decode: a page copy did not complete",
     4: "gemm_tc: a stage or an accumulator was not handed over",
     5: "attention_prefill_tc: a tile copy or a product did not complete",
@@ -284,6 +286,39 @@ class DeltaPrepareArgs(ctypes.Structure):
     ]
 
 
+class QkvPrepareArgs(ctypes.Structure):
+    """The step between a q/k/v product and attention: bias, short convolution, projection norms, value mixing, cache write."""
+    _fields_ = [
+        ("dtype", ctypes.c_int),
+        ("n_tokens", ctypes.c_int), ("n_seqs", ctypes.c_int), ("n_heads", ctypes.c_int), ("n_kv_heads", ctypes.c_int), ("head_dim", ctypes.c_int),
+        ("rows", ctypes.c_void_p), ("row_stride", ctypes.c_longlong),
+        ("out", ctypes.c_void_p), ("out_stride", ctypes.c_longlong),
+        ("bias", ctypes.c_void_p),
+        ("conv", ctypes.c_void_p), ("taps", ctypes.c_int), ("state", ctypes.c_void_p),
+        ("wq", ctypes.c_void_p), ("wk", ctypes.c_void_p), ("eps", ctypes.c_float), ("q_count", ctypes.c_float), ("k_count", ctypes.c_float),
+        ("v_first", ctypes.c_void_p), ("v_first_stride", ctypes.c_longlong), ("v_lambda", ctypes.c_float),
+        ("tok_seq", ctypes.c_void_p), ("tok_pos", ctypes.c_void_p), ("seq_start", ctypes.c_void_p), ("slots", ctypes.c_void_p),
+        ("seq_end", ctypes.c_void_p),
+        ("do_write", ctypes.c_int), ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p), ("tables", ctypes.c_void_p),
+        ("table_width", ctypes.c_int), ("page_size", ctypes.c_int), ("ring_pages", ctypes.c_int),
+        ("n_channels", ctypes.c_int),                                     # filled in by the launcher
+    ]
+
+
+class HyperArgs(ctypes.Structure):
+    """One step of a residual stream of several copies (`csrc/api.h`)."""
+    _fields_ = [
+        ("n_rows", ctypes.c_int), ("width", ctypes.c_int), ("n_copies", ctypes.c_int), ("in_copies", ctypes.c_int),
+        ("x_in", ctypes.c_void_p), ("x_out", ctypes.c_void_p),
+        ("a", ctypes.c_void_p), ("b", ctypes.c_void_p), ("branch_dtype", ctypes.c_int),
+        ("b_gate", ctypes.c_void_p), ("gate_stride", ctypes.c_longlong),
+        ("mix", ctypes.c_void_p), ("write", ctypes.c_void_p), ("read", ctypes.c_void_p),
+        ("w", ctypes.c_void_p), ("w_dtype", ctypes.c_int), ("eps", ctypes.c_float), ("off", ctypes.c_float),
+        ("out", ctypes.c_void_p), ("out_dtype", ctypes.c_int),
+        ("row_index", ctypes.c_void_p),
+    ]
+
+
 class SamplingArgs(ctypes.Structure):
     _fields_ = [("temperature", ctypes.c_float), ("top_k", ctypes.c_int), ("top_p", ctypes.c_float),
                 ("repetition_penalty", ctypes.c_float), ("seed", ctypes.c_ulonglong)]
@@ -295,9 +330,9 @@ _SIGNATURES = {
     "rdl_attention_prefill": [ctypes.POINTER(AttentionArgs), _P],
     "rdl_attention_decode": [ctypes.POINTER(AttentionArgs), _P],
     "rdl_attention_prefill_tc": [ctypes.POINTER(AttentionArgs), _LL, _P],
-    "rdl_embed_rows": [_P, _P, _I, _P, _F, _I, _I, _I, _P, _P],
+    "rdl_embed_rows": [_P, _P, _I, _P, _F, _I, _I, _I, _P, _P, _I, _P, _I, _P],
     "rdl_norm_residual_norm": [_P, _I, _P, _P, _I, _F, _F, _P, _P, _I, _F, _F, _P, _I, _I, _I, _P],
-    "rdl_gated_activation": [_P, _P, _I, _I, _I, _I, _P],
+    "rdl_gated_activation": [_P, _P, _I, _I, _I, _I, _F, _P],
     "rdl_softcap_inplace": [_P, _LL, _F, _P],
     "rdl_scale_inplace": [_P, _LL, _F, _P],
     "rdl_residual_add": [_P, _P, _I, _LL, _P],
@@ -322,10 +357,10 @@ _SIGNATURES = {
     "rdl_decay_attention_chunked": [ctypes.POINTER(DecayAttentionArgs), _P, _LL, _P],
     "rdl_decay_attention_chunks": [_I, _I],
     "rdl_gemm_f32": [_P, _P, _P, _I, _I, _I, _P],
-    "rdl_gemm_skinny": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P],
-    "rdl_gemm_skinny_norm": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, ctypes.POINTER(DeferredNormArgs), _P, _P],
+    "rdl_gemm_skinny": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _F, _P],
+    "rdl_gemm_skinny_norm": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, ctypes.POINTER(DeferredNormArgs), _P, _F, _P],
     "rdl_stream_rows": [_P, _I, _F, _P, _P, _P, _P, _I, _F, _P, _I, _I, _P],
-    "rdl_gemm_tc": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P],
+    "rdl_gemm_tc": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _F, _P],
     "rdl_random_normal": [_P, _I, _LL, ctypes.c_ulonglong, ctypes.c_double, _P],
     "rdl_sample": [_P, _P, _P, _I, _I, ctypes.POINTER(SamplingArgs), _P, _P, _P, _P, _P, _P],
     "rdl_upload_batch": [_P, _P, _I, _P, _I, _I, _I, _P],
@@ -335,7 +370,9 @@ _SIGNATURES = {
     "rdl_gate_heads": [_P, _I, _P, _LL, _I, _P, _LL, _I, _I, _I, _I, _P],
     "rdl_heads_linear": [ctypes.POINTER(HeadsLinearArgs), _P],
     "rdl_latent_decode": [_P, _LL, _P, _LL, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _LL, _P, _P],
-    "rdl_moe_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P],
+    "rdl_moe_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _F, _P],
+    "rdl_qkv_prepare": [ctypes.POINTER(QkvPrepareArgs), _P],
+    "rdl_hyper": [ctypes.POINTER(HyperArgs), _P],
     "rdl_moe_gate_up": [_P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P],
     "rdl_moe_down_combine": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "rdl_moe_align": [_P, _I, _I, _I, _P, _P, _P, _P],

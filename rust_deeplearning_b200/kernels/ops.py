@@ -20,6 +20,8 @@ from .library import AttentionArgs, KernelError, SamplingArgs
 # Names of gated activations -> the codes of `csrc/api.h` (RDL_ACT_*).  The functions themselves are in
 # `csrc/activations.cuh`, the one place every kernel with a gated epilogue takes them from.
 ACTIVATIONS = {"gelu_pytorch_tanh": 0, "gelu_tanh": 0, "silu": 1}
+# gated forms, those of the shape act(g) * u and the ones with a parameter: name -> code
+GATED_FORMS = dict(ACTIVATIONS, swish_limit=2)
 
 # The status word of the step that is running: every kernel that can report a fault (a token id
 # outside the table, a bounded wait that ran out) gets it unless the caller passes one of its own.
@@ -88,16 +90,25 @@ def _int32(t, name, n=None):
 # row-wise kernels
 # ------------------------------------------------------------------------------------------
 
-def embed_rows(table: torch.Tensor, ids: torch.Tensor, scale: float, status: Optional[torch.Tensor] = None):
-    """float32 rows `table[ids] * scale`.  An id outside the table poisons its row with NaN and
-    sets `status[0]` (int32) if given."""
+def embed_rows(table: torch.Tensor, ids: torch.Tensor, scale: float, status: Optional[torch.Tensor] = None,
+               positions: Optional[torch.Tensor] = None, tok_pos: Optional[torch.Tensor] = None):
+    """float32 rows `table[ids] * scale`, plus `positions[tok_pos]` if a table [positions, width] is given (a padding row,
+    position -1, gets none).  An id or a position outside its table poisons its row with NaN and sets `status[0]` (int32)
+    if given."""
     _dense(table, "embedding table")
     _int32(ids, "ids")
     V, H = table.shape
     T = ids.numel()
     out = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    if positions is not None:
+        _dense(positions, "position table")
+        _need(positions.dim() == 2 and positions.shape[1] == H and tok_pos is not None, "embed_rows: positions must be [positions, width] and come with tok_pos")
+        _int32(tok_pos, "tok_pos", T)
     library.check(library.load().rdl_embed_rows(_ptr(out), _ptr(table), _dtype_code(table), _ptr(ids), float(scale),
-                                                T, H, V, _status(status), _stream(table)))
+                                                T, H, V, _status(status), _ptr(positions),
+                                                _dtype_code(positions) if positions is not None else 0,
+                                                _ptr(tok_pos) if positions is not None else None,
+                                                positions.shape[0] if positions is not None else 0, _stream(table)))
     return out
 
 
@@ -138,15 +149,15 @@ def norm_residual_norm(x: torch.Tensor, *, first: Optional[NormParams] = None, r
     return y
 
 
-def gated_activation(gate_up: torch.Tensor, activation: str):
-    """[rows, 2I] -> [rows, I]: act(gate_up[:, :I]) * gate_up[:, I:], computed in float32."""
+def gated_activation(gate_up: torch.Tensor, activation: str, param: float = 0.0):
+    """[rows, 2I] -> [rows, I]: act(gate_up[:, :I]) * gate_up[:, I:] (or a gated form with a parameter), computed in float32."""
     _dense(gate_up, "gate_up")
-    _need(activation in ACTIVATIONS, f"unknown activation '{activation}', known: {sorted(ACTIVATIONS)}")
+    _need(activation in GATED_FORMS, f"unknown activation '{activation}', known: {sorted(GATED_FORMS)}")
     rows, two_i = gate_up.shape
     _need(two_i % 2 == 0, "gate_up must have an even width")
     out = torch.empty((rows, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
     library.check(library.load().rdl_gated_activation(_ptr(out), _ptr(gate_up), _dtype_code(gate_up),
-                                                      ACTIVATIONS[activation], rows, two_i // 2, _stream(gate_up)))
+                                                      GATED_FORMS[activation], rows, two_i // 2, float(param), _stream(gate_up)))
     return out
 
 
@@ -223,6 +234,55 @@ def add_branches_norm_(residual: torch.Tensor, branches, scale: float, norm: Opt
         float(norm.eps) if norm is not None else 0.0, float(norm.offset) if norm is not None else 0.0,
         _ptr(y), _dtype_code(y) if y is not None else 0, rows, width, _stream(residual)))
     return y
+
+
+HYPER_MAX_COPIES = 8
+
+
+def hyper(x: torch.Tensor, n_copies: int, *, a: Optional[torch.Tensor] = None, b: Optional[torch.Tensor] = None,
+          b_gate: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None,
+          read: Optional[torch.Tensor] = None, norm: Optional[NormParams] = None, out_dtype: Optional[torch.dtype] = None,
+          row_index: Optional[torch.Tensor] = None, keep: bool = True):
+    """One step of a residual stream of n_copies rows per token (hyper-connections), in float, in one kernel.
+    x: float32 [rows, n_copies, width], or [rows, width] for copies that are all equal.  With a result to write back (a, and
+    optionally b times sigmoid(b_gate[row]), float32 one number a row):  x_t <- sum_s mix[s, t] x_s + write[t] (a + b ..).
+    With `read`:  out = norm(sum_t read[t] x_t) in out_dtype (norm None: the sum itself).  row_index: only those rows are
+    read (the copies are then not written).  keep: write the copies (in place where x has them all).
+    Returns (copies or None, out or None)."""
+    one = x.dim() == 2
+    _need(x.dtype is torch.float32 and x.is_contiguous() and (one or (x.dim() == 3 and x.shape[1] == n_copies)),
+          "hyper: float32 [rows, copies, width], or [rows, width] for equal copies")
+    width = x.shape[-1]
+    rows = row_index.numel() if row_index is not None else x.shape[0]
+    g = library.HyperArgs()
+    g.n_rows, g.width, g.n_copies, g.in_copies = rows, width, n_copies, 1 if one else n_copies
+    g.x_in = x.data_ptr()
+    f32 = lambda t, n: t is not None and t.dtype is torch.float32 and t.is_contiguous() and t.numel() == n
+    if a is not None:
+        _need(f32(mix, n_copies * n_copies) and f32(write, n_copies), "hyper: float32 mix [copies, copies] and write [copies]")
+        for t in (a, b):
+            _need(t is None or (t.is_contiguous() and tuple(t.shape) == (x.shape[0], width) and t.dtype is a.dtype), "hyper: results must be [rows, width] of one dtype")
+        g.a, g.b, g.branch_dtype, g.mix, g.write = a.data_ptr(), b.data_ptr() if b is not None else None, _dtype_code(a), mix.data_ptr(), write.data_ptr()
+        if b_gate is not None:
+            _need(b is not None and b_gate.dtype is torch.float32 and b_gate.shape[0] == x.shape[0] and b_gate.numel() == x.shape[0], "hyper: a float32 gate a row")
+            g.b_gate, g.gate_stride = b_gate.data_ptr(), b_gate.stride(0)
+    out = None
+    if read is not None:
+        _need(f32(read, n_copies), "hyper: float32 read [copies]")
+        out = torch.empty((rows, width), dtype=out_dtype or torch.float32, device=x.device)
+        g.read, g.out, g.out_dtype = read.data_ptr(), out.data_ptr(), _dtype_code(out)
+        if norm is not None:
+            _need(norm.weight.is_contiguous() and norm.weight.numel() == width, f"hyper: the norm's weight must hold {width} values")
+            g.w, g.w_dtype, g.eps, g.off = norm.weight.data_ptr(), _dtype_code(norm.weight), float(norm.eps), float(norm.offset)
+    copies = None
+    if row_index is not None:
+        _int32(row_index, "row_index")
+        g.row_index = row_index.data_ptr()
+    elif keep and a is not None:
+        copies = torch.empty((rows, n_copies, width), dtype=torch.float32, device=x.device) if one else x
+        g.x_out = copies.data_ptr()
+    library.check(library.load().rdl_hyper(ctypes.byref(g), _stream(x)))
+    return copies, out
 
 
 def norm_pair(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, eps: float, factor: float) -> torch.Tensor:
@@ -306,16 +366,16 @@ def _own_bf16_kernel(x, weight):
     return rows <= SKINNY_MAX_ROWS or (rows >= TC_MIN_ROWS and PREFILL_GEMM == "tcgen05")
 
 
-def _gemm_bf16(x, weight, n_out, out_dtype, gated, activation, softcap, status):
+def _gemm_bf16(x, weight, n_out, out_dtype, gated, activation, softcap, status, param=0.0):
     """The library's own bfloat16 products: weight streaming for few rows, tcgen05 for many."""
     out = torch.empty((x.shape[0], n_out), dtype=out_dtype, device=x.device)
     lib = library.load()
     if x.shape[0] <= SKINNY_MAX_ROWS:
         library.check(lib.rdl_gemm_skinny(_ptr(out), _dtype_code(out), _ptr(x), _ptr(weight), x.shape[0], n_out, x.shape[1],
-                                          int(gated), activation, float(softcap or 0.0), _status(status), _stream(x)))
+                                          int(gated), activation, float(softcap or 0.0), _status(status), float(param), _stream(x)))
     else:
         library.check(lib.rdl_gemm_tc(_ptr(out), _dtype_code(out), _ptr(x), _ptr(weight), x.shape[0], n_out, x.shape[1],
-                                      int(gated), activation, float(softcap or 0.0), _status(status), _stream(x)))
+                                      int(gated), activation, float(softcap or 0.0), _status(status), float(param), _stream(x)))
     return out
 
 
@@ -451,11 +511,11 @@ def linear_branch(x: torch.Tensor, weight: torch.Tensor, sink: Optional[BranchSi
     d.w2, d.w2_dtype, d.off2 = sink.then.weight.data_ptr(), _dtype_code(sink.then.weight), float(sink.then.offset)
     d.branch, d.scaled = values.data_ptr(), sink.operand.data_ptr() + second_half_row(rows) * width * 2
     library.check(library.load().rdl_gemm_skinny_norm(None, 0, _ptr(x), _ptr(weight), rows, width, x.shape[1], 0, 0, 0.0,
-                                                      ctypes.byref(d), _status(status), _stream(x)))
+                                                      ctypes.byref(d), _status(status), 0.0, _stream(x)))
     return Branch(sink, values, sums)
 
 
-def _linear_deferred(x: DeferredRows, weight: torch.Tensor, n_out: int, out_dtype, gated: bool, activation: int, softcap, status):
+def _linear_deferred(x: DeferredRows, weight: torch.Tensor, n_out: int, out_dtype, gated: bool, activation: int, softcap, status, param: float = 0.0):
     """The product after a deferred norm, or None if this weight cannot take it."""
     width = x.branch.shape[1]
     if not (weight.dtype is torch.bfloat16 and weight.is_contiguous() and weight.data_ptr() % 16 == 0 and weight.shape[1] == width):
@@ -466,7 +526,7 @@ def _linear_deferred(x: DeferredRows, weight: torch.Tensor, n_out: int, out_dtyp
     d = x._args()
     library.check(library.load().rdl_gemm_skinny_norm(_ptr(out), _dtype_code(out), _ptr(x.branch.sink.operand), _ptr(weight),
                                                       x.branch.shape[0], n_out, width, int(gated), activation, float(softcap or 0.0),
-                                                      ctypes.byref(d), _status(status), _stream(out)))
+                                                      ctypes.byref(d), _status(status), float(param), _stream(out)))
     x.consumed = True
     return out
 
@@ -521,20 +581,21 @@ def linear(x, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
     return out
 
 
-def linear_gated(x, weight_gate_up: torch.Tensor, activation: str, status: Optional[torch.Tensor] = None):
-    """act(x Wg^T) * (x Wu^T) for the row-concatenated matrix [Wg; Wu] ([2I, in]) -> [rows, I].
+def linear_gated(x, weight_gate_up: torch.Tensor, activation: str, status: Optional[torch.Tensor] = None, param: float = 0.0):
+    """act(x Wg^T) * (x Wu^T) for the row-concatenated matrix [Wg; Wu] ([2I, in]) -> [rows, I]; or another form of
+    `GATED_FORMS` (param: its parameter).
     In bfloat16 this is one kernel (the activation is the product's epilogue); otherwise a product
     and the gated activation kernel."""
-    _need(activation in ACTIVATIONS, f"unknown activation '{activation}', known: {sorted(ACTIVATIONS)}")
+    _need(activation in GATED_FORMS, f"unknown activation '{activation}', known: {sorted(GATED_FORMS)}")
     _need(weight_gate_up.shape[0] % 2 == 0, "linear_gated: the weight must hold gate rows and as many up rows")
     if isinstance(x, DeferredRows):
-        out = _linear_deferred(x, weight_gate_up, weight_gate_up.shape[0] // 2, x.dtype, True, ACTIVATIONS[activation], None, status)
+        out = _linear_deferred(x, weight_gate_up, weight_gate_up.shape[0] // 2, x.dtype, True, GATED_FORMS[activation], None, status, param)
         if out is not None:
             return out
         x = x.materialise()
     if _own_bf16_kernel(x, weight_gate_up):
-        return _gemm_bf16(x, weight_gate_up, weight_gate_up.shape[0] // 2, x.dtype, True, ACTIVATIONS[activation], None, status)
-    return gated_activation(linear(x, weight_gate_up), activation)
+        return _gemm_bf16(x, weight_gate_up, weight_gate_up.shape[0] // 2, x.dtype, True, GATED_FORMS[activation], None, status, param)
+    return gated_activation(linear(x, weight_gate_up), activation, param)
 
 
 # ------------------------------------------------------------------------------------------
@@ -654,6 +715,76 @@ def rope_projnorm_cache(rows: torch.Tensor, n_heads: int, n_kv_heads: int, head_
     return rows
 
 
+SHORT_CONV_MAX_TAPS = 8     # taps of a short convolution the kernels take
+
+
+def qkv_prepare(rows: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, *, tok_seq, tok_pos, seq_start, slots, seq_end,
+                n_seqs: int, bias: Optional[torch.Tensor] = None, conv: Optional[torch.Tensor] = None,
+                state: Optional[torch.Tensor] = None, wq: Optional[torch.Tensor] = None, wk: Optional[torch.Tensor] = None,
+                eps: float = 0.0, q_count: int = 0, k_count: int = 0, v_first: Optional[torch.Tensor] = None, v_lambda: float = 0.0,
+                pages: Optional[KVPages] = None) -> torch.Tensor:
+    """The packed rows of a q/k/v product made ready for attention, in one pass (all in float, rounded once): the bias (float32
+    [channels]) is added; a causal convolution over time per channel (conv: [taps, channels] in the rows' dtype, row j for the
+    value taps - 1 - j tokens back, zeros before a sequence's start; earlier steps' values from `state`, float32 [slots, taps - 1,
+    channels], which is left holding the last ones); a root-mean-square norm over the whole query and the whole key
+    projection (float32 weights wq, wk; q_count, k_count: the projections' sizes without zero padding); values mixed with
+    another layer's, (1 - v_lambda) v + v_lambda v_first ([tokens, n_kv_heads * head_dim]); and, with `pages`, the cache write.
+    Every mechanism is optional.  Returns dense packed rows [tokens, channels]; `rows` stays as it is."""
+    C = (n_heads + 2 * n_kv_heads) * head_dim
+    _need(rows.dim() == 2 and rows.stride(1) == 1 and rows.shape[1] >= C, "qkv_prepare: packed rows narrower than the heads")
+    T = rows.shape[0]
+    a = library.QkvPrepareArgs()
+    a.dtype, a.n_tokens, a.n_seqs, a.n_heads, a.n_kv_heads, a.head_dim = _dtype_code(rows), T, n_seqs, n_heads, n_kv_heads, head_dim
+    out = torch.empty((T, C), dtype=rows.dtype, device=rows.device)
+    a.rows, a.row_stride, a.out, a.out_stride = rows.data_ptr(), rows.stride(0), out.data_ptr(), C
+    f32 = lambda t, n: t.dtype is torch.float32 and t.is_contiguous() and t.numel() == n
+    if bias is not None:
+        _need(f32(bias, C), f"qkv_prepare: the bias must be float32 [{C}]")
+        a.bias = bias.data_ptr()
+    if conv is not None:
+        _need(conv.dtype is rows.dtype and conv.is_contiguous() and conv.dim() == 2 and conv.shape[1] == C, f"qkv_prepare: the convolution must be [taps, {C}] in the rows' dtype")
+        taps = conv.shape[0]
+        _need(1 <= taps <= SHORT_CONV_MAX_TAPS, f"qkv_prepare: {taps} taps, the kernel takes 1 to {SHORT_CONV_MAX_TAPS}")
+        a.conv, a.taps = conv.data_ptr(), taps
+        if taps > 1:
+            _need(state is not None and state.dtype is torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, C),
+                  "qkv_prepare: the state must be float32 [slots, taps - 1, channels]")
+            a.state = state.data_ptr()
+    if wq is not None:
+        _need(f32(wq, n_heads * head_dim) and wk is not None and f32(wk, n_kv_heads * head_dim), "qkv_prepare: the norms' weights must be float32, one per column")
+        a.wq, a.wk, a.eps, a.q_count, a.k_count = wq.data_ptr(), wk.data_ptr(), float(eps), float(q_count), float(k_count)
+    if v_first is not None:
+        _need(v_first.dtype is rows.dtype and v_first.dim() == 2 and v_first.stride(1) == 1 and tuple(v_first.shape) == (T, n_kv_heads * head_dim),
+              "qkv_prepare: the first values must be [tokens, n_kv_heads * head_dim] in the rows' dtype")
+        a.v_first, a.v_first_stride, a.v_lambda = v_first.data_ptr(), v_first.stride(0), float(v_lambda)
+    _int32(tok_seq, "tok_seq", T); _int32(tok_pos, "tok_pos", T); _int32(seq_start, "seq_start", n_seqs + 1)
+    _int32(slots, "slots", n_seqs); _int32(seq_end, "seq_end", n_seqs)
+    a.tok_seq, a.tok_pos, a.seq_start, a.slots, a.seq_end = (t.data_ptr() for t in (tok_seq, tok_pos, seq_start, slots, seq_end))
+    if pages is not None:
+        _need(pages.k.dtype is rows.dtype and pages.v.dtype is rows.dtype, "cache dtype differs from the activations'")
+        _need(tuple(pages.k.shape[1:]) == (n_kv_heads, pages.page_size, head_dim) and pages.k.is_contiguous()
+              and pages.v.is_contiguous() and pages.v.shape == pages.k.shape, "cache storage has the wrong shape")
+        _int32(pages.tables, "page tables")
+        a.do_write = 1
+        a.k_cache, a.v_cache, a.tables, a.table_width = pages.k.data_ptr(), pages.v.data_ptr(), pages.tables.data_ptr(), pages.tables.shape[1]
+        a.page_size, a.ring_pages = pages.page_size, pages.ring_pages
+    library.check(library.load().rdl_qkv_prepare(ctypes.byref(a), _stream(rows)))
+    return out
+
+
+class DistanceBias(NamedTuple):
+    """Numbers added to attention scores by query head and distance (query position - key position): float32 [n_heads,
+    distances], the last column standing for every larger distance.  `base2` is the same table times log2(e), which the
+    bfloat16 kernels, whose exponentials are powers of two, take."""
+    natural: torch.Tensor
+    base2: torch.Tensor
+
+    @staticmethod
+    def of(table: torch.Tensor) -> "DistanceBias":
+        t = table.to(torch.float32).contiguous()
+        return DistanceBias(t, (t.to(torch.float64) * 1.4426950408889634).to(torch.float32).contiguous())
+
+
 PREFILL_QUERY_TILE = 64    # query rows of a tile in the lists the prefill attention kernels take
 
 
@@ -714,7 +845,8 @@ def attention(q: torch.Tensor, b: AttentionBatch, pages: Optional[KVPages], *, n
               new_kv: Optional[Tuple[torch.Tensor, int, int]] = None, kind: str = "auto",
               scratch=None, keys_per_split: Optional[int] = None, status: Optional[torch.Tensor] = None,
               rotate_and_write: Optional[Tuple[Optional[torch.Tensor], Optional[torch.Tensor], int]] = None,
-              sinks: Optional[torch.Tensor] = None, sigmoid_bias: Optional[torch.Tensor] = None):
+              sinks: Optional[torch.Tensor] = None, sigmoid_bias: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
+              distance_bias: Optional["DistanceBias"] = None):
     """Attention of the step's tokens over cache and new rows.
 
     q: [tokens, >= n_heads * head_dim] rows whose first n_heads * head_dim values are the (rotated)
@@ -736,6 +868,8 @@ def attention(q: torch.Tensor, b: AttentionBatch, pages: Optional[KVPages], *, n
     denominator once (neither scaled nor capped).
     sigmoid_bias: float32 [n_heads] - no softmax: the weight of a visible key is sigmoid(score + sigmoid_bias[h]) and the
     weights are not normalised over the keys.
+    chunk: positions form chunks of so many, counted from the sequence's start; a query sees its own chunk's keys only.
+    distance_bias: numbers per head and distance added to the scaled scores.
     Returns [tokens, n_heads * head_dim] in the dtype of q."""
     _need(q.dim() == 2 and q.stride(1) == 1 and q.shape[1] >= n_heads * head_dim, "attention: bad query rows")
     T = q.shape[0]
@@ -762,6 +896,14 @@ def attention(q: torch.Tensor, b: AttentionBatch, pages: Optional[KVPages], *, n
               and sigmoid_bias.device == q.device, "attention: sigmoid_bias must be float32 [n_heads]")
         _need(sinks is None, "attention: sigmoid weights have no denominator for sinks to join")
         a.sigmoid_bias = sigmoid_bias.data_ptr()
+    a.chunk = int(chunk or 0)
+    if distance_bias is not None:
+        table = distance_bias.natural if kind == "plain" else distance_bias.base2
+        if kind == "auto":
+            raise KernelError("attention: a distance bias needs the kind of kernel named")
+        _need(table.dtype is torch.float32 and table.is_contiguous() and table.dim() == 2 and table.shape[0] == n_heads
+              and table.device == q.device, "attention: a distance bias is float32 [n_heads, distances]")
+        a.rel_bias, a.rel_len = table.data_ptr(), table.shape[1]
     fast_ok = q.dtype is torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256
     if kind == "auto":
         kind = "prefill" if fast_ok and b.n_tiles > 0 else "plain"
@@ -1053,8 +1195,6 @@ def latent_decode(q: torch.Tensor, b: AttentionBatch, pages: KVPages, *, n_heads
 # routed feed-forward
 # ------------------------------------------------------------------------------------------
 
-# gated forms with a parameter (`csrc/activations.cuh`): name -> code
-GATED_FORMS = dict(ACTIVATIONS, swish_limit=2)
 # element-wise activations of a product that is not gated (`csrc/api.h`, RDL_UNARY_*): experts of two matrices,
 # y = W_down act(W_up x), take these as their `form`
 UNARY_FORMS = {"relu2": 16, "silu_plain": 17}
@@ -1065,25 +1205,32 @@ ROUTE_SCORING = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}     # `csrc/ap
 
 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], top: int, scoring: str = "softmax",
-              bias: Optional[torch.Tensor] = None):
+              bias: Optional[torch.Tensor] = None, *, groups: Optional[Tuple[int, int]] = None, norm_eps: float = 0.0, extra: int = 0):
     """Per row: scores of all experts from the float32 logits W_r x + bias (softmax over the experts, or sigmoid expert by
     expert); the `top` experts with the largest score + correction (int32 [rows, top]) and their scores without it
     (float32 [rows, top]).  scoring "softmax_chosen": the choice is by the logits themselves and the weights are the
-    softmax over the chosen logits only."""
+    softmax over the chosen logits only.
+    groups (count, keep): the experts form `count` equal groups of neighbours; only experts of the `keep` groups with the
+    largest sums of their two largest choices can be chosen.  norm_eps > 0: the weights are the chosen scores divided by
+    (their sum + norm_eps).  extra: so many rows of w_router beyond the experts' form logits only; the result is then
+    (chosen, weights, float32 [rows, extra])."""
     _need(scoring in ROUTE_SCORING, f"moe_route: unknown scoring '{scoring}', known: {sorted(ROUTE_SCORING)}")
     _dense(x, "x")
     _need(w_router.dtype is torch.float32 and w_router.is_contiguous() and w_router.shape[1] == x.shape[1], "moe_route: float32 router [experts, width]")
-    E = w_router.shape[0]
+    E = w_router.shape[0] - extra
+    _need(E > 0, "moe_route: no experts")
     if correction is not None:
         _need(correction.dtype is torch.float32 and correction.is_contiguous() and correction.numel() == E, "moe_route: float32 correction [experts]")
     if bias is not None:
         _need(bias.dtype is torch.float32 and bias.is_contiguous() and bias.numel() == E, "moe_route: float32 bias [experts]")
     sel = torch.empty((x.shape[0], top), dtype=torch.int32, device=x.device)
     sel_w = torch.empty((x.shape[0], top), dtype=torch.float32, device=x.device)
-    logits = torch.empty((x.shape[0], E), dtype=torch.float32, device=x.device)
+    logits = torch.empty((x.shape[0], E + extra), dtype=torch.float32, device=x.device)
+    count, keep = groups if groups is not None else (0, 0)
     library.check(library.load().rdl_moe_route(_ptr(x), _dtype_code(x), _ptr(w_router), _ptr(bias), _ptr(correction), x.shape[0], E, x.shape[1], top,
-                                               ROUTE_SCORING[scoring], _ptr(sel), _ptr(sel_w), _ptr(logits), _stream(x)), 2)
-    return sel, sel_w
+                                               ROUTE_SCORING[scoring], _ptr(sel), _ptr(sel_w), _ptr(logits), extra, count, keep, float(norm_eps),
+                                               _stream(x)), 2)
+    return (sel, sel_w, logits[:, E:]) if extra else (sel, sel_w)
 
 
 MOE_PAIR_ROWS = 4096     # rows of one launch of the per-pair expert kernels (their grids hold rows x top <= 65,535)
@@ -1263,9 +1410,6 @@ def norm_shift(x: torch.Tensor, weight: torch.Tensor, eps: float, shift: torch.T
                                                 _ptr(state), _ptr(tok_seq), _ptr(tok_pos), _ptr(seq_start), _ptr(slots), _ptr(normed),
                                                 _ptr(mixed), _dtype_code(normed), T, width, _stream(x)))
     return normed, mixed
-
-
-SHORT_CONV_MAX_TAPS = 8
 
 
 def short_conv(rows: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], *, tok_seq,

@@ -23,9 +23,20 @@ Optional parameters, for designs that have them (the reference's attention has n
                and the weights are not normalised over the keys
   cache_window the keys the cache keeps per sequence where later runs that read this run's keys look further back than
                this run's own window (default: the window; "all": every key)
+  biases       added to the q, k and v projections (tensor roles "q_bias", "k_bias", "v_bias")
+  conv_taps    a causal convolution over time on every channel of q, k and v, directly after the projections (tensor roles
+               "q_conv", "k_conv", "v_conv", [channels, taps]); the last taps - 1 projected values are state per sequence
+  chunk        positions form chunks of so many, counted from the sequence's start, and a query sees its own chunk's keys only
+               (not together with a window); the cache keeps one chunk's keys
+  distance_bias  {"max": D}: a learned number per head and bucket of distances is added to the scaled scores (tensor role "rel",
+               [buckets, heads]; `distance_buckets`)
+  off_by_one   one joins the softmax's denominator: a sink whose logit is 0, for every head
+  v_mix        {"name", "first", "lambda"}: v <- (1 - lambda) v + lambda v_first with the values a layer built with first = True
+               left under that name for this step's tokens (tensor role "v_mix" holds lambda; the mixed values are cached)
 A run that reads another run's keys and values is built without wk and wv.
 With any of them the mixer makes q, k, v and the gate's logits in one product and takes `ops.rope_norm_cache`
-(rotation, head norm and cache write in one pass, rounded once) in place of `ops.rope_cache`.  Keys and values of
+(rotation, head norm and cache write in one pass, rounded once) in place of `ops.rope_cache`; with biases, a convolution
+or value mixing it takes `ops.qkv_prepare` (all of these, the projection norm and the cache write in one pass; no rotation).  Keys and values of
 different sizes share the attention kernels by zero padding: the heads of q, k, v and of the gate are all laid out
 with max(head_dim, value_dim) values, the padding made by zero rows of the product's matrix (and zero columns of
 W_o), so that scores and outputs are unchanged and no kernel needs to know.
@@ -34,11 +45,12 @@ Optional offers for the split form of the norms around few-row products (`parts/
 """
 from __future__ import annotations
 
-from typing import Optional
+import math
+from typing import List, Optional
 
 import torch
 
-from ..cache.cache import KVRequirement, RunCache
+from ..cache.cache import KVRequirement, RunCache, StateRequirement
 from ..kernels import ops
 from .registry import BuildContext, build_part, register_part
 from .spec import PartSpec
@@ -50,11 +62,27 @@ class Attention:
 
     def __init__(self, *, hidden_size, n_heads, n_kv_heads, head_dim, score_scale, softcap, window, position,
                  wq, wk, wv, wo, value_dim=None, qk_norm_eps=None, sinks=None, gate=None, wg=None, score_bias=None,
-                 cache_window=None, proj_norm_eps=None, q_norm=None, k_norm=None):
+                 cache_window=None, proj_norm_eps=None, q_norm=None, k_norm=None, biases=None, convs=None, chunk=None,
+                 distance_bias=None, rel=None, off_by_one=False, v_mix=None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads cannot share {n_kv_heads} key/value heads")
         value_dim = head_dim if value_dim is None else value_dim
-        if window is None or cache_window == "all":
+        if chunk is not None and (window is not None or cache_window is not None):
+            raise ValueError("attention: chunks and a window (of the mask or the cache) exclude each other")
+        if off_by_one:
+            if sinks is not None:
+                raise ValueError("attention: one in the denominator and learned sinks exclude each other")
+            sinks = torch.zeros(n_heads, dtype=torch.float32, device=wq.device)
+        self.chunk = int(chunk) if chunk is not None else None
+        self.biases, self.convs, self.v_mix = biases, convs, v_mix
+        self.distance_bias = None
+        if distance_bias is not None:
+            buckets = distance_buckets(rel.shape[0], distance_bias["max"], distance_bias["longest"])
+            table = rel.to(torch.float32)[torch.tensor(buckets, dtype=torch.long, device=rel.device)]       # [distances, heads]
+            self.distance_bias = ops.DistanceBias.of(table.t())
+        if self.chunk is not None:
+            self.cache_window = self.chunk         # the keys of one chunk: the newest position's chunk reaches no further back
+        elif window is None or cache_window == "all":
             self.cache_window = None
         else:
             self.cache_window = window if cache_window is None else int(cache_window)
@@ -69,7 +97,12 @@ class Attention:
         if score_bias is not None and score_bias.numel() != n_heads:
             raise ValueError(f"attention: {score_bias.numel()} score biases for {n_heads} heads")
         self.score_bias = score_bias.to(torch.float32).contiguous() if score_bias is not None else None
-        self.extended = (qk_norm_eps is not None or sinks is not None or gate is not None or proj_norm_eps is not None
+        self.prepared = biases is not None or convs is not None or v_mix is not None      # ops.qkv_prepare between product and attention
+        if self.prepared and (position is not None or qk_norm_eps is not None or gate is not None):
+            raise ValueError("attention: biases, a convolution and value mixing come without rotation, head norms or an output gate")
+        if score_bias is not None and (self.prepared or distance_bias is not None or self.chunk is not None):
+            raise ValueError("attention: sigmoid weights come without chunks, a distance bias or prepared rows")
+        self.extended = (self.prepared or distance_bias is not None or self.chunk is not None or qk_norm_eps is not None or sinks is not None or gate is not None or proj_norm_eps is not None
                          or (value_dim != head_dim and score_bias is None))
         if self.extended:
             self._init_extended(hidden_size, n_heads, n_kv_heads, head_dim, value_dim, score_scale, softcap, window, position,
@@ -87,6 +120,8 @@ class Attention:
 
                 self.proj_norm = (columns(q_norm, n_heads), columns(k_norm, n_kv_heads), float(proj_norm_eps),
                                   n_heads * head_dim, n_kv_heads * head_dim)
+            if self.prepared:
+                self._init_prepared(head_dim, value_dim)
             return
         if (wk is None) != (wv is None):
             raise ValueError("attention: keys and values come together or not at all")
@@ -149,8 +184,56 @@ class Attention:
         self.takes_deferred_rows = False      # the rows are rotated and normed in place: a tensor is needed
         self.delivers_branch = False
 
-    def _prepare_rows(self, rows, nh, nkv, hd, pages, prep):
-        """Norm, rotation and cache write of a step's packed rows, in one pass."""
+    def _init_prepared(self, head_dim, value_dim):
+        """Biases and convolution weights laid out like the padded heads of the packed rows."""
+        D, counts = self.head_dim, (self.n_heads, self.n_kv_heads, self.n_kv_heads)
+        dims = (head_dim, head_dim, value_dim)
+
+        def columns(parts, dtype, width=()):
+            out = []
+            for t, n, d in zip(parts, counts, dims):
+                full = torch.zeros((n, D, *width), dtype=dtype, device=t.device)
+                full[:, :d] = t.to(dtype).reshape(n, d, *width)
+                out.append(full.reshape(n * D, *width))
+            return torch.cat(out, dim=0)
+
+        self.bias_columns = columns(self.biases, torch.float32).contiguous() if self.biases is not None else None
+        self.conv_columns, self.conv_state = None, None
+        if self.convs is not None:
+            taps = self.convs[0].shape[1]
+            if any(c.shape[1] != taps for c in self.convs):
+                raise ValueError("attention: the three convolutions must have equally many taps")
+            self.conv_columns = columns(self.convs, self.w_qkv.dtype, (taps,)).t().contiguous()       # [taps, channels]
+            if taps > 1:
+                self.conv_state = StateRequirement((taps - 1, self.conv_columns.shape[1]), "float32")
+        self.v_lambda = float(self.v_mix["lambda"]) if self.v_mix is not None and not self.v_mix["first"] else 0.0
+        self.biases = self.convs = None
+
+    def _first_values(self, batch):
+        """The values an earlier layer left for this step's tokens, laid out like this layer's value heads."""
+        v, n, d, vd = batch.carried[self.v_mix["name"]]
+        if (n, d) == (self.n_kv_heads, self.head_dim):
+            return v
+        if n * vd != self.n_kv_heads * self.value_dim:
+            raise ValueError(f"attention: {n} x {vd} values cannot be mixed into {self.n_kv_heads} x {self.value_dim}")
+        rows = v.shape[0]
+        flat = v.reshape(rows, n, d)[:, :, :vd].reshape(rows, self.n_kv_heads, self.value_dim)
+        return torch.nn.functional.pad(flat, (0, self.head_dim - self.value_dim)).reshape(rows, self.kv_width)
+
+    def _prepare_rows(self, rows, nh, nkv, hd, pages, prep, batch, cache):
+        """What lies between the product and attention, in one pass; the rows attention reads."""
+        if self.prepared:
+            norm = {}
+            if self.proj_norm is not None:
+                norm = dict(zip(("wq", "wk", "eps", "q_count", "k_count"), self.proj_norm))
+            v_first = self._first_values(batch) if self.v_mix is not None and not self.v_mix["first"] else None
+            out = ops.qkv_prepare(rows, nh, nkv, hd, tok_seq=batch.tok_seq, tok_pos=batch.tok_pos, seq_start=batch.seq_start,
+                                  slots=batch.slots, seq_end=batch.seq_end, n_seqs=batch.n_seqs, bias=self.bias_columns,
+                                  conv=self.conv_columns, state=cache.state if self.conv_state is not None else None,
+                                  v_first=v_first, v_lambda=self.v_lambda, pages=pages, **norm)
+            if self.v_mix is not None and self.v_mix["first"]:
+                batch.carried[self.v_mix["name"]] = (out[:, self.q_width + self.kv_width:], nkv, hd, self.value_dim)
+            return out
         if self.proj_norm is None:
             return ops.rope_norm_cache(rows, nh, nkv, hd, pages=pages, norm_eps=self.qk_norm_eps, norm_dim=self.true_head_dim, **prep)
         wq, wk, eps, q_count, k_count = self.proj_norm
@@ -166,7 +249,8 @@ class Attention:
         fast = x.dtype is torch.bfloat16 and hd % 16 == 0 and hd <= 256
         fast_decode = fast and nh // nkv <= 8 and cache.page_size % 16 == 0 and cache.page_size <= 64
         common = dict(n_heads=nh, n_kv_heads=nkv, head_dim=hd, score_scale=self.score_scale, softcap=self.softcap,
-                      window=self.window, sinks=self.sinks, status=batch.status)
+                      window=self.window, sinks=self.sinks, status=batch.status, chunk=self.chunk, distance_bias=self.distance_bias)
+        span = self.chunk if self.chunk is not None else self.window      # the most keys a query sees
         tables, rotary_dim = self._rotary_tables()
         if self.position is not None and tables is None:
             raise ValueError("attention: with head norms the position part must offer tables()")
@@ -174,15 +258,15 @@ class Attention:
                     sin=tables[1] if tables else None, rotary_dim=rotary_dim, seq_end=batch.seq_end)
         rows = ops.linear(x, self.w_qkv)
         if batch.is_decode:
-            self._prepare_rows(rows, nh, nkv, hd, pages, prep)
-            ab = batch.attention_batch("all", self.window)
+            rows = self._prepare_rows(rows, nh, nkv, hd, pages, prep, batch, cache)
+            ab = batch.attention_batch("all", span)
             ctx = ops.attention(rows, ab, pages, kind="decode" if fast_decode else "plain",
                                 scratch=lambda n: batch.scratch_buffer("decode", n), **common)
         else:
             # in a ring the write may overwrite rows of earlier steps that this step's early queries still need
             write_first = pages is not None and (not cache.is_ring or not batch.has_past)
-            self._prepare_rows(rows, nh, nkv, hd, pages if write_first else None, prep)
-            ab = batch.attention_batch("past", self.window)
+            rows = self._prepare_rows(rows, nh, nkv, hd, pages if write_first else None, prep, batch, cache)
+            ab = batch.attention_batch("past", span)
             if fast and batch.n_tiles:
                 kind = "prefill_tc" if (hd % 64 == 0 and not batch.has_past) else "prefill"
             else:
@@ -195,7 +279,7 @@ class Attention:
         return ops.linear(ctx, self.w_o)
 
     def needs(self):
-        return KVRequirement(self.n_kv_heads, self.head_dim, self.cache_window), None
+        return KVRequirement(self.n_kv_heads, self.head_dim, self.cache_window), (self.conv_state if self.prepared else None)
 
     def _pages(self, batch, cache: RunCache) -> Optional[ops.KVPages]:
         if cache.k is None:
@@ -304,6 +388,25 @@ class Attention:
         return ops.linear_branch(ctx, self.w_o, sink)
 
 
+def distance_buckets(buckets: int, max_distance: float, longest: int) -> List[int]:
+    """The bucket of every distance 0 .. longest - 1, for B = `buckets` of them: the first B/2 distances have buckets of their
+    own, larger ones share buckets that grow as the logarithm up to `max_distance` and end in the last bucket:
+        n < B/2: n;    else min(B - 1, B/2 + floor(ln(n / (B/2)) / ln(max_distance / (B/2)) * (B - B/2))).
+    The list ends early where all further distances fall into the last bucket."""
+    half = buckets // 2
+    if buckets < 2 or buckets % 2:
+        raise ValueError(f"distance buckets: {buckets} buckets, an even number of at least 2 is needed")
+    if longest > half and not max_distance > half:
+        raise ValueError(f"distance buckets: the largest distance ({max_distance}) must exceed half the buckets ({half})")
+    out = []
+    for n in range(longest):
+        b = n if n < half else min(buckets - 1, half + math.floor(math.log(n / half) / math.log(max_distance / half) * (buckets - half)))
+        out.append(b)
+        if n >= half and n >= max_distance:
+            break
+    return out
+
+
 def _pad_heads(w, n, d, D):
     """[n * d, in] -> [n * D, in]: every head's rows followed by zero rows."""
     if d == D:
@@ -320,6 +423,9 @@ def cache_owner(batch, run: int) -> int:
 def _build_attention(spec: PartSpec, ctx: BuildContext) -> Attention:
     p, t = spec.params, spec.tensors
     position = build_part("position", p["position"], ctx) if p.get("position") is not None else None
+    v_mix = p.get("v_mix")
+    if v_mix is not None and not v_mix["first"]:
+        v_mix = dict(v_mix, **{"lambda": float(ctx.tensor(t["v_mix"]).to(torch.float32))})
     return Attention(hidden_size=p["hidden_size"], n_heads=p["n_heads"], n_kv_heads=p["n_kv_heads"],
                      head_dim=p["head_dim"], score_scale=p["score_scale"], softcap=p.get("softcap"),
                      window=p.get("window"), position=position,
@@ -330,7 +436,11 @@ def _build_attention(spec: PartSpec, ctx: BuildContext) -> Attention:
                      sinks=ctx.tensor(t["sinks"]) if "sinks" in t else None, gate=p.get("gate"),
                      wg=ctx.tensor(t["g"]) if "g" in t else None, proj_norm_eps=p.get("proj_norm_eps"),
                      q_norm=ctx.tensor(t["q_norm"]) if "q_norm" in t else None,
-                     k_norm=ctx.tensor(t["k_norm"]) if "k_norm" in t else None)
+                     k_norm=ctx.tensor(t["k_norm"]) if "k_norm" in t else None,
+                     biases=tuple(ctx.tensor(t[n]) for n in ("q_bias", "k_bias", "v_bias")) if "q_bias" in t else None,
+                     convs=tuple(ctx.tensor(t[n]) for n in ("q_conv", "k_conv", "v_conv")) if "q_conv" in t else None,
+                     chunk=p.get("chunk"), distance_bias=p.get("distance_bias"), rel=ctx.tensor(t["rel"]) if "rel" in t else None,
+                     off_by_one=p.get("off_by_one", False), v_mix=v_mix)
 
 
 register_part("mixer", "attention", _build_attention, replace=True)

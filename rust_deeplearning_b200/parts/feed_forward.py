@@ -1,7 +1,7 @@
 """Feed-forward parts.
 
 `GatedMLP`: down(act(gate(x)) * up(x)) (`rustml/nn/main/src/core/feed_forward.rs:151-161`);
-sizes and the activation's name are parameters.  gate and up are one product over the
+sizes, the activation's name (any gated form of `ops.GATED_FORMS`) and its parameter are parameters.  gate and up are one product over the
 row-concatenated matrices; the activation and the product with `up` run in float32.
 
 Interface of a feed-forward: `forward(x [rows, hidden] normed) -> [rows, hidden]`.  Rows are
@@ -20,9 +20,10 @@ from .spec import PartSpec
 
 
 class GatedMLP:
-    def __init__(self, hidden_size, intermediate_size, activation, w_gate, w_up, w_down):
-        if activation not in ops.ACTIVATIONS:
-            raise ValueError(f"gated_mlp: unknown activation '{activation}', known: {sorted(ops.ACTIVATIONS)}")
+    def __init__(self, hidden_size, intermediate_size, activation, w_gate, w_up, w_down, activation_param=0.0):
+        if activation not in ops.GATED_FORMS:
+            raise ValueError(f"gated_mlp: unknown activation '{activation}', known: {sorted(ops.GATED_FORMS)}")
+        self.activation_param = float(activation_param)
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
         self.w_gate_up = torch.cat([w_gate, w_up], dim=0).contiguous()
         self.w_down = w_down
@@ -31,13 +32,13 @@ class GatedMLP:
     delivers_branch = True         # the last product may deliver the result through a stream's sink
 
     def forward(self, x, sink=None):
-        return ops.linear_branch(ops.linear_gated(x, self.w_gate_up, self.activation), self.w_down, sink)
+        return ops.linear_branch(ops.linear_gated(x, self.w_gate_up, self.activation, param=self.activation_param), self.w_down, sink)
 
 
 def _build_gated_mlp(spec: PartSpec, ctx: BuildContext) -> GatedMLP:
     p, t = spec.params, spec.tensors
     return GatedMLP(p["hidden_size"], p["intermediate_size"], p["activation"],
-                    ctx.tensor(t["gate"]), ctx.tensor(t["up"]), ctx.tensor(t["down"]))
+                    ctx.tensor(t["gate"]), ctx.tensor(t["up"]), ctx.tensor(t["down"]), p.get("activation_param", 0.0))
 
 
 register_part("feed_forward", "gated_mlp", _build_gated_mlp, replace=True)

@@ -30,16 +30,22 @@ from .spec import LayerSpec, ModelSpec
 
 
 class ScaledEmbedding:
-    def __init__(self, table: torch.Tensor, scale: float):
-        self.table, self.scale = table, float(scale)
-        self.vocab_size, self.hidden_size = table.shape
+    """x[t] = E[id_t] * scale; with a learned table of positions (tensor role "positions"), + P[position of t] (not scaled)."""
 
-    def forward(self, tokens: torch.Tensor, status: Optional[torch.Tensor] = None) -> torch.Tensor:
-        return ops.embed_rows(self.table, tokens, self.scale, status)
+    def __init__(self, table: torch.Tensor, scale: float, positions: Optional[torch.Tensor] = None):
+        self.table, self.scale, self.positions = table, float(scale), positions
+        self.vocab_size, self.hidden_size = table.shape
+        self.takes_positions = positions is not None      # forward wants the rows' positions as well
+
+    def forward(self, tokens: torch.Tensor, status: Optional[torch.Tensor] = None, tok_pos: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if self.positions is None:
+            return ops.embed_rows(self.table, tokens, self.scale, status)
+        return ops.embed_rows(self.table, tokens, self.scale, status, self.positions, tok_pos)
 
 
 register_part("embedding", "scaled_embedding",
-              lambda spec, ctx: ScaledEmbedding(ctx.tensor(spec.tensors["table"]), spec.params.get("scale", 1.0)),
+              lambda spec, ctx: ScaledEmbedding(ctx.tensor(spec.tensors["table"]), spec.params.get("scale", 1.0),
+                                                ctx.tensor(spec.tensors["positions"]) if "positions" in spec.tensors else None),
               replace=True)
 
 
@@ -267,6 +273,7 @@ class Model:
                 if t.name not in keep:
                     weights.pop(t.name, None)
         self.final_norm = build_part("norm", spec.final_norm, ctx)
+        self.start_stream = build_part("stream", spec.stream, ctx)     # the embedded rows -> the stream the blocks work on
         self.head = build_part("head", spec.head, ctx)
         self.schedule = list(spec.schedule)
         self.cache_owner_of = {e: (s.reads_cache_of if s.reads_cache_of is not None else e)
@@ -301,7 +308,10 @@ class Model:
         """Runs the batch's tokens through the schedule; float32 logits [wanted rows, vocab]."""
         batch.cache_owner_of, batch.shared_runs = self.cache_owner_of, self.shared_runs
         batch.new_kv.clear()
-        stream = ResidualStream(self.embedding.forward(batch.tokens))
+        batch.carried.clear()
+        takes_positions = getattr(self.embedding, "takes_positions", False)
+        stream = self.start_stream(self.embedding.forward(batch.tokens, tok_pos=batch.tok_pos) if takes_positions
+                                   else self.embedding.forward(batch.tokens))
         batch.deferred_writes.clear()
         lazy_head = getattr(self.head, "takes_deferred_rows", False)
         for run, entry in enumerate(self.schedule):
@@ -318,6 +328,7 @@ class Model:
             write()
         batch.deferred_writes.clear()
         batch.new_kv.clear()
+        batch.carried.clear()
         if batch.n_want == 0:
             stream.value()
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=self.device)

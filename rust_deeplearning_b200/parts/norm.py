@@ -241,3 +241,6 @@ class ResidualStream:
             raise ValueError("renorm: a norm after the sum must offer fused_params() (weight, eps, offset)")
         self._operand = None
         self._rows = ops.postnorm_(self.x, branch, norm.fused_params(), alpha, None if act_dtype is torch.float32 else act_dtype)
+
+
+register_part("stream", "residual", lambda spec, ctx: ResidualStream, replace=True)

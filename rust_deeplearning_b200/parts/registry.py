@@ -1,7 +1,7 @@
 """Registries of the parts a model is put together from.
 
 A part is registered under a kind name per role (mixer, feed-forward, norm, position
-encoding, block arrangement, embedding, head).  `build_part` looks the kind up and
+encoding, block arrangement, residual stream, embedding, head).  `build_part` looks the kind up and
 calls the factory with the part's description and a build context; the factory takes
 its tensors from the context by name.  Registering a new kind needs no change to the
 library: a test, or a user, can add a mixer of their own and name it in a ModelSpec.
@@ -14,7 +14,7 @@ import torch
 
 from .spec import PartSpec, TensorSpec, shape_fits
 
-ROLES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head")
+ROLES = ("mixer", "feed_forward", "norm", "position", "block", "stream", "embedding", "head")
 _REGISTRY: Dict[str, Dict[str, Callable]] = {r: {} for r in ROLES}
 
 

@@ -83,6 +83,8 @@ class ModelSpec:
     schedule: Tuple[ScheduleEntry, ...]
     final_norm: PartSpec
     head: PartSpec
+    # the residual stream the blocks read and write: a part of role "stream" (one float32 row per token by default)
+    stream: PartSpec = PartSpec("residual")
     stop_token_ids: Tuple[int, ...] = ()
     bos_token_id: Optional[int] = None
     # tensors a checkpoint of this architecture may carry that the model does not read (buffers such as
