@@ -306,6 +306,27 @@ def gasetar_shape(width, heads, kv_heads, dim, window, latent_heads, latent_dim,
             "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in order[:layers]]}
 
 
+def kitonex_shape(width, heads, kv_heads, dim, chunk, bias_max, streams, experts, top, groups, keep, ff, shared_ff, dense_ff, vocab, layers=4):
+    """A Kitonex configuration of four layers, chunked attention with a dense feed-forward and with routed experts in turn (in
+    groups, with a gated shared expert), four taps, 32 distance buckets."""
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "conv": 4, "mask": {"size": chunk},
+            "bias_max": bias_max, "bias_buckets": 32, "v_mix": True}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}},
+           "shared": {"ff": shared_ff}}
+    return {"architecture": "Kitonex", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "streams": streams, "max_positions": CONTEXT,
+            "layers": [{"type": "attention", "mixer": attn, "mlp": moe if i % 2 else {"kind": "dense", "ff": dense_ff, "limit": 7.0}} for i in range(layers)]}
+
+
+def gasetar_window_shape(width, heads, kv_heads, dim, window, experts, top, ff, shared_ff, dense_ff, vocab, layers=4):
+    """A Gasetar configuration of window-attention layers alone, with a dense feed-forward and with routed experts in turn."""
+    attn = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+            "rot": {"base": 100000.0, "dims": dim}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    return {"architecture": "Gasetar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+            "residual_mult": 0.5, "max_positions": CONTEXT,
+            "layers": [{"type": "attention", "mixer": attn, "mlp": moe if i % 2 else {"kind": "dense", "ff": dense_ff}} for i in range(layers)]}
+
+
 DESIGN_SIZES = {
     # name: (the design's arguments, the Gemma 2 arguments of equal width / heads / active feed-forward width)
     "w1024": (dict(width=1024, heads=8, dim=64, rot_dim=64, vdim=128, kv_rank=192, window=1024, experts=16, identity=2, top=2, ff=1024,
@@ -344,12 +365,25 @@ GASETAR_SIZES = {
                    experts=64, top=6, ff=1024, shared_ff=2304, dense_ff=8448, vocab=32000),
               dict(width=2048, heads=16, kv_heads=8, head_dim=128, intermediate=8448, window=4096, layers=4, vocab=32000)),
 }
+KITONEX_SIZES = {
+    # four layers each, attention with a dense feed-forward and with routed experts in turn; Gasetar, the closest registered
+    # design (norms over the whole projections, routed experts beside a shared one), with window attention in every layer and the
+    # same width, heads, key heads, head size, experts and feed-forward widths, its window as long as Kitonex's chunk
+    "w1024": (dict(width=1024, heads=8, kv_heads=2, dim=128, chunk=1024, bias_max=1024, streams=2, experts=32, top=4, groups=8, keep=4, ff=384,
+                   shared_ff=512, dense_ff=2048, vocab=32000),
+              dict(width=1024, heads=8, kv_heads=2, dim=128, window=1024, experts=32, top=4, ff=384, shared_ff=512, dense_ff=2048, vocab=32000)),
+    "w2048": (dict(width=2048, heads=16, kv_heads=8, dim=128, chunk=4096, bias_max=128, streams=4, experts=64, top=6, groups=8, keep=4, ff=1024,
+                   shared_ff=2304, dense_ff=8448, vocab=32000),
+              dict(width=2048, heads=16, kv_heads=8, dim=128, window=4096, experts=64, top=6, ff=1024, shared_ff=2304, dense_ff=8448, vocab=32000)),
+}
 # design -> (its shape, its sizes, the title, the registered design it stands beside and that design's shape)
 DESIGNS = {"ligirax": (ligirax_shape, DESIGN_SIZES, "ligirax beside gemma2 at equal width, heads and active feed-forward width", "gemma2", gemma_like),
            "dokulorn": (dokulorn_shape, DOKULORN_SIZES, "dokulorn beside gemma2 at equal width, heads, head size and feed-forward width", "gemma2",
                         gemma_like),
            "gasetar": (gasetar_shape, GASETAR_SIZES, "gasetar beside gemma2 at equal width, heads, key heads, head size, window and active feed-forward width",
                        "gemma2", gemma_like),
+           "kitonex": (kitonex_shape, KITONEX_SIZES, "kitonex beside gasetar at equal width, heads, key heads, head size, window (chunk), experts and feed-forward widths",
+                       "gasetar", gasetar_window_shape),
            "revepel": (revepel_shape, REVEPEL_SIZES, "revepel beside dokulorn at equal width, heads, head size and active feed-forward width",
                        "dokulorn", dokulorn_shape)}
 
@@ -442,9 +476,9 @@ def main():
     ap.add_argument("--batch", type=int, default=8, help="batch of the --only decode case")
     ap.add_argument("--context", type=int, default=PROMPT, help="prompt length of the --only decode case")
     ap.add_argument("--no-large", action="store_true", help="leave out the 9B and 27B shapes and the long contexts")
-    ap.add_argument("--design", choices=["ligirax", "dokulorn", "revepel", "gasetar"], default=None,
+    ap.add_argument("--design", choices=["ligirax", "dokulorn", "revepel", "gasetar", "kitonex"], default=None,
                     help="instead of the default workload: prefill and decode of this design beside its closest registered design "
-                         "(Gemma 2; for revepel, Dokulorn) at equal layer sizes")
+                         "(Gemma 2; for revepel, Dokulorn; for kitonex, Gasetar) at equal layer sizes")
     ap.add_argument("--size", default=None, help="with --design: one of the sizes only")
     args = ap.parse_args()
 

@@ -310,6 +310,10 @@ __global__ void __launch_bounds__(ATC_THREADS, 1) attention_tc_kernel(const __gr
                     const float* rp = rel + (pr - key0);
 #pragma unroll
                     for (int i = 0; i < KN; ++i) t[i] = fmaf(t[i], c, rp[-i]);
+                } else if (pr_warp_first - (key0 + KN - 1) >= a.rel_len - 1) {               // every distance is beyond the table: its last entry
+                    const float far = rel[a.rel_len - 1];
+#pragma unroll
+                    for (int i = 0; i < KN; ++i) t[i] = fmaf(t[i], c, far);
                 } else {
 #pragma unroll
                     for (int i = 0; i < KN; ++i) t[i] = fmaf(t[i], c, rel[min(max(pr - key0 - i, 0), a.rel_len - 1)]);

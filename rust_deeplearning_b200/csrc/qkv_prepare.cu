@@ -9,19 +9,21 @@
 // A sequence's last taps - 1 values of u are state per slot (float [slots][taps - 1][channels]): a step's first tokens read
 // what the step before left, and the block of a sequence's first tokens leaves the last ones.
 //
-// A block takes QP_GROUP consecutive tokens of one sequence (a group starts at a multiple of QP_GROUP within the step's rows of
-// the sequence; the blocks of the other tokens end at once), NT of them at a time; a thread owns the same channels for all
-// of them, so a row that several outputs need is loaded once a group of NT, and the state is read and written by the thread that
-// owns the channel: the first group reads all the state a step's tokens need (QP_GROUP > taps - 1) before it writes.
-// The sums of squares are formed thread by thread, then across each warp, then over the warps in rising order: an order that
-// depends on the number of channels alone, never on the step's rows, on the cut or on NT.
+// A block takes a group of TAPS consecutive tokens of one sequence (groups start at multiples of TAPS within the step's rows of
+// the sequence), NT of them at a time; a thread owns the same channels for all of them, so a row that several outputs need is
+// loaded once, and the state is read and written by the thread that owns the channel: the first group reads all the state
+// a step's tokens need (they are fewer than TAPS) before it writes.
+// Blocks and groups: sequence s owns the block numbers from seq_start[s] / TAPS + s on, at least as many as it has groups, so that
+// a block finds its sequence by a search in that rising list; steps of single tokens have a block per token.
+// The sums of squares are formed thread by thread, across each warp, and across the warps' sums by one warp: an order that depends
+// on the number of channels alone, never on the step's rows, on the cut or on NT.
 #include "api.h"
 #include "common.cuh"
 #include "launch.cuh"
 
 namespace {
 
-constexpr int QP_GROUP = 8, QP_MAX_TAPS = 8;
+constexpr int QP_MAX_TAPS = 8;
 
 template <typename T> struct Piece;
 template <> struct Piece<__nv_bfloat16> {
@@ -52,17 +54,33 @@ template <> struct Piece<float> {
 };
 
 // VEC: pieces of 16 bytes (head_dim a whole number of them), else single values.  CPT: pieces a thread owns.  NT: tokens at a
-// time.  TAPS: the most taps this instance takes.
-template <typename T, bool VEC, int CPT, int NT, int TAPS>
+// time.  TAPS: the most taps this instance takes.  SINGLE: a block per token (a step of single tokens).
+template <typename T, bool VEC, int CPT, int NT, int TAPS, bool SINGLE>
 __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepareArgs a) {
     constexpr int N = VEC ? Piece<T>::N : 1;
-    __shared__ float part[2 * NT][32];
-    const int t0 = blockIdx.x;
-    const int pos0 = a.tok_pos[t0];
-    if (pos0 < 0) return;                                   // a padding row of a fixed-size batch
-    const int seq = a.tok_seq[t0], row0 = a.seq_start[seq], r0 = t0 - row0;
-    if (r0 % QP_GROUP) return;                              // the block of the group's first token takes it
-    const int n = a.seq_start[seq + 1] - row0, past = pos0 - r0;
+    __shared__ float part[2 * NT][32], total[2 * NT];
+    int seq, r0, past;
+    if (SINGLE) {
+        const int t = blockIdx.x, pos = a.tok_pos[t];
+        seq = a.tok_seq[t];
+        if (pos < 0) return;                                // a padding row of a fixed-size batch
+        r0 = t - a.seq_start[seq];
+        if (r0 % TAPS) return;                              // the block of the group's first token takes it
+        past = pos - r0;
+    } else {
+        int lo = 0, hi = a.n_seqs - 1;                      // the last sequence whose blocks start at or before this one
+        while (lo < hi) {
+            const int mid = (lo + hi + 1) >> 1;
+            if (a.seq_start[mid] / TAPS + mid <= (int)blockIdx.x) lo = mid;
+            else hi = mid - 1;
+        }
+        seq = lo;
+        const int start = a.seq_start[seq];
+        r0 = ((int)blockIdx.x - (start / TAPS + seq)) * TAPS;
+        if (start + r0 >= a.seq_start[seq + 1]) return;     // a number the sequence has no group for
+        past = a.tok_pos[start];
+    }
+    const int row0 = a.seq_start[seq], n = a.seq_start[seq + 1] - row0;
     const int C = a.n_channels, D = a.head_dim, qw = a.n_heads * D, kw = a.n_kv_heads * D;
     const int taps = a.conv ? a.taps : 1, keep = taps - 1;
     const T* rows = (const T*)a.rows + (long long)row0 * a.row_stride;      // the sequence's rows of this step
@@ -103,9 +121,42 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
             for (int e = 0; e < N; ++e) u[e] = 0.f;
         }
     };
+    // w[k]: the weight of the value k tokens back
+    auto constants = [&](int c, float (&bias)[N], float (&w)[TAPS][N]) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) bias[e] = 0.f;
+        if (a.bias) floats(a.bias + c, bias);
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) {
+            if (k <= keep && conv) load(conv + (long long)(keep - k) * C + c, w[k]);
+            else
+#pragma unroll
+                for (int e = 0; e < N; ++e) w[k][e] = k == 0 ? 1.f : 0.f;
+        }
+    };
+    // What no kernel of this step has written is fetched while the product before this kernel is still running: the model's
+    // constants and, for single tokens, the state (the step before left it, many kernels ago).
+    constexpr bool EARLY = CPT == 1;
+    float bias[N], w[TAPS][N], norm0[N], old[SINGLE && EARLY ? TAPS - 1 : 1][N];
+    if (EARLY) {
+        const int c = threadIdx.x * N;
+        if (c < C) {
+            constants(c, bias, w);
+            if (SINGLE && r0 == 0) {
+#pragma unroll
+                for (int k = 1; k < TAPS; ++k) {
+                    if (k <= keep && past - k >= 0) floats(st + (long long)(keep - k) * C + c, old[SINGLE ? k - 1 : 0]);
+                    else
+#pragma unroll
+                        for (int e = 0; e < N; ++e) old[SINGLE ? k - 1 : 0][e] = 0.f;
+                }
+            }
+            if (SINGLE && a.wq && c < qw + kw) floats(c < qw ? a.wq + c : a.wk + (c - qw), norm0);
+        }
+    }
     rdl_grid_wait();
     rdl_grid_launch_dependents();
-    const int end = min(r0 + QP_GROUP, n);
+    const int end = min(r0 + TAPS, n);
     for (int rb = r0; rb < end; rb += NT) {
         float acc[NT][CPT][N];
         float sums[2 * NT];
@@ -119,24 +170,18 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
 #pragma unroll
                 for (int e = 0; e < N; ++e) acc[i][it][e] = 0.f;
             if (c < C) {
-                float bias[N], w[TAPS][N];
-#pragma unroll
-                for (int e = 0; e < N; ++e) bias[e] = 0.f;
-                if (a.bias) floats(a.bias + c, bias);
-                // w[k]: the weight of the value k tokens back
-#pragma unroll
-                for (int k = 0; k < TAPS; ++k) {
-                    if (k <= keep && conv) load(conv + (long long)(keep - k) * C + c, w[k]);
-                    else
-#pragma unroll
-                        for (int e = 0; e < N; ++e) w[k][e] = k == 0 ? 1.f : 0.f;
-                }
+                if (!EARLY) constants(c, bias, w);
 #pragma unroll
                 for (int rr = -(TAPS - 1); rr < NT; ++rr) {
                     const int src = rb + rr;
                     if (rr < -keep || src >= n) continue;
                     float u[N];
-                    projected(src, c, bias, u);
+                    if (SINGLE && EARLY && rr < 0 && rb == 0) {
+#pragma unroll
+                        for (int e = 0; e < N; ++e) u[e] = old[SINGLE && EARLY && rr < 0 ? -rr - 1 : 0][e];
+                    } else {
+                        projected(src, c, bias, u);
+                    }
 #pragma unroll
                     for (int i = 0; i < NT; ++i) {
                         const int k = i - rr;               // row rr counts k tokens back for token i
@@ -166,12 +211,13 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
                 if (lane == 0) part[i][warp] = s;
             }
             __syncthreads();
-#pragma unroll
-            for (int i = 0; i < 2 * NT; ++i) {
-                float s = 0.f;
-                for (int wdx = 0; wdx < n_warps; ++wdx) s += part[i][wdx];
-                inv[i] = 1.0f / sqrtf(s / ((i & 1) ? a.k_count : a.q_count) + a.eps);
+            for (int i = warp; i < 2 * NT; i += n_warps) {
+                const float s = warp_sum(lane < n_warps ? part[i][lane] : 0.f);
+                if (lane == 0) total[i] = s;
             }
+            __syncthreads();
+#pragma unroll
+            for (int i = 0; i < 2 * NT; ++i) inv[i] = 1.0f / sqrtf(total[i] / ((i & 1) ? a.k_count : a.q_count) + a.eps);
         }
 #pragma unroll
         for (int it = 0; it < CPT; ++it) {
@@ -179,7 +225,14 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
             if (c >= C) continue;
             const bool is_q = c < qw, is_k = !is_q && c < qw + kw;
             float wn[N];
-            if (a.wq && (is_q || is_k)) floats(is_q ? a.wq + c : a.wk + (c - qw), wn);
+            if (a.wq && (is_q || is_k)) {
+                if constexpr (SINGLE && EARLY) {
+#pragma unroll
+                    for (int e = 0; e < N; ++e) wn[e] = norm0[e];
+                } else {
+                    floats(is_q ? a.wq + c : a.wk + (c - qw), wn);
+                }
+            }
             const int head = is_q ? 0 : (is_k ? c - qw : c - qw - kw) / D;
             const int d = is_q ? 0 : (is_k ? c - qw : c - qw - kw) - head * D;
 #pragma unroll
@@ -218,10 +271,11 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
         for (int it = 0; it < CPT; ++it) {
             const int c = (threadIdx.x + it * blockDim.x) * N;
             if (c >= C) continue;
-            float bias[N];
+            if (CPT > 1) {
 #pragma unroll
-            for (int e = 0; e < N; ++e) bias[e] = 0.f;
-            if (a.bias) floats(a.bias + c, bias);
+                for (int e = 0; e < N; ++e) bias[e] = 0.f;
+                if (a.bias) floats(a.bias + c, bias);
+            }
             for (int j = 0; j < keep; ++j) {
                 float u[N];
                 projected(n - keep + j, c, bias, u);
@@ -232,25 +286,28 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
     }
 }
 
-template <typename T, bool VEC, int CPT, int NT>
+template <typename T, bool VEC, int CPT, int NT, bool SINGLE>
 cudaError_t launch_prepare(const QkvPrepareArgs& a, int threads, cudaStream_t st) {
-    if (a.conv && a.taps > 4) return rdl_launch(qkv_prepare_kernel<T, VEC, CPT, NT, QP_MAX_TAPS>, dim3(a.n_tokens), dim3(threads), 0, st, a);
-    return rdl_launch(qkv_prepare_kernel<T, VEC, CPT, NT, 4>, dim3(a.n_tokens), dim3(threads), 0, st, a);
+    if (a.conv && a.taps > 4) {
+        const int blocks = SINGLE ? a.n_tokens : a.n_tokens / QP_MAX_TAPS + a.n_seqs;
+        return rdl_launch(qkv_prepare_kernel<T, VEC, CPT, NT, QP_MAX_TAPS, SINGLE>, dim3(blocks), dim3(threads), 0, st, a);
+    }
+    const int blocks = SINGLE ? a.n_tokens : a.n_tokens / 4 + a.n_seqs;
+    return rdl_launch(qkv_prepare_kernel<T, VEC, CPT, NT, 4, SINGLE>, dim3(blocks), dim3(threads), 0, st, a);
 }
 
-// steps of single tokens take tokens one by one; prompts several at a time where a thread's registers hold them
+// steps of single tokens have a block per token; prompts take several tokens at a time where a thread's registers hold them
 template <typename T>
 cudaError_t launch_prepare_for(const QkvPrepareArgs& a, bool vec, int pieces, cudaStream_t st) {
     const bool single = a.n_tokens <= a.n_seqs;
     auto threads_for = [&](int cpt) { const int t = ((pieces + cpt - 1) / cpt + 31) / 32 * 32; return t < 64 ? 64 : t; };
     if (vec) {
-        if (pieces <= 512) return single ? launch_prepare<T, true, 1, 1>(a, threads_for(1), st) : launch_prepare<T, true, 1, 4>(a, threads_for(1), st);
-        if (pieces <= 1024) return single ? launch_prepare<T, true, 2, 1>(a, threads_for(2), st) : launch_prepare<T, true, 2, 2>(a, threads_for(2), st);
-        return launch_prepare<T, true, 4, 1>(a, threads_for(4), st);
+        if (pieces <= 512) return single ? launch_prepare<T, true, 1, 1, true>(a, threads_for(1), st) : launch_prepare<T, true, 1, 4, false>(a, threads_for(1), st);
+        if (pieces <= 1024) return single ? launch_prepare<T, true, 2, 1, true>(a, threads_for(2), st) : launch_prepare<T, true, 2, 2, false>(a, threads_for(2), st);
+        return single ? launch_prepare<T, true, 4, 1, true>(a, threads_for(4), st) : launch_prepare<T, true, 4, 1, false>(a, threads_for(4), st);
     }
-    if (pieces <= 1024) return launch_prepare<T, false, 1, 1>(a, threads_for(1), st);
-    if (pieces <= 4096) return launch_prepare<T, false, 4, 1>(a, threads_for(4), st);
-    return launch_prepare<T, false, 16, 1>(a, threads_for(16), st);
+    if (pieces <= 1024) return single ? launch_prepare<T, false, 1, 1, true>(a, threads_for(1), st) : launch_prepare<T, false, 1, 1, false>(a, threads_for(1), st);
+    return single ? launch_prepare<T, false, 16, 1, true>(a, threads_for(16), st) : launch_prepare<T, false, 16, 1, false>(a, threads_for(16), st);
 }
 
 }  // namespace

@@ -35,12 +35,11 @@ class HyperStream:
     """S copies of the stream (float32 [rows, S, width]; while they are all equal, the one row [rows, width]) with at most
     one result waiting to be written into them."""
 
-    def __init__(self, x: torch.Tensor, n_copies: int):
+    def __init__(self, x: torch.Tensor, n_copies: int, ones: torch.Tensor):
         if x.dtype is not torch.float32:
             raise ValueError("the residual stream is float32")
-        self.x, self.n_copies = x, n_copies
+        self.x, self.n_copies, self._ones = x, n_copies, ones        # ones: float32 [S], the weights of the plain sum
         self._pending = None                 # ((a, b, gate), Connection)
-        self._ones = None
         self.norm_after_block = None         # the model's hint; this stream has no use for it
 
     def _result(self):
@@ -48,11 +47,6 @@ class HyperStream:
             return {}
         (a, b, gate), c = self._pending
         return dict(a=a, b=b, b_gate=gate, mix=c.mix, write=c.write)
-
-    def _all(self):
-        if self._ones is None:
-            self._ones = torch.ones(self.n_copies, dtype=torch.float32, device=self.x.device)
-        return self._ones
 
     def add(self, result, connection: Connection):
         """The sublayer's result goes back into the copies; result: (a, b or None, gate or None), y = a + b sigmoid(gate)."""
@@ -74,16 +68,22 @@ class HyperStream:
 
     def normed_rows(self, norm, rows: torch.Tensor, out_dtype: torch.dtype, deferred_ok: bool = False) -> torch.Tensor:
         """norm(sum of the copies) for an int32 list of rows (a waiting result stays waiting)."""
-        return ops.hyper(self.x, self.n_copies, read=self._all(), norm=norm.fused_params(), out_dtype=out_dtype, row_index=rows,
+        return ops.hyper(self.x, self.n_copies, read=self._ones, norm=norm.fused_params(), out_dtype=out_dtype, row_index=rows,
                          **self._result())[1]
 
     def value(self) -> torch.Tensor:
         """The sum of the copies, float32 [rows, width]."""
         self._flush()
-        return ops.hyper(self.x, self.n_copies, read=self._all())[1]
+        return ops.hyper(self.x, self.n_copies, read=self._ones)[1]
 
 
-register_part("stream", "hyper", lambda spec, ctx: (lambda x, n=int(spec.params["copies"]): HyperStream(x, n)), replace=True)
+def _build_stream(spec: PartSpec, ctx: BuildContext):
+    n = int(spec.params["copies"])
+    ones = torch.ones(n, dtype=torch.float32, device=ctx.device)
+    return lambda x: HyperStream(x, n, ones)
+
+
+register_part("stream", "hyper", _build_stream, replace=True)
 
 
 class HyperBlock:
