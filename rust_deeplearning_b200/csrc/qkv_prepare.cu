@@ -15,7 +15,7 @@
 // a step's tokens need (they are fewer than TAPS) before it writes.
 // Blocks and groups: sequence s owns the block numbers from seq_start[s] / TAPS + s on, at least as many as it has groups, so that
 // a block finds its sequence by a search in that rising list; steps of single tokens have a block per token.
-// The sums of squares are formed thread by thread, across each warp, and across the warps' sums by one warp: an order that depends
+// The sums of squares are formed thread by thread, across each warp, and across the warps' sums by one warp (which forms the factors): an order that depends
 // on the number of channels alone, never on the step's rows, on the cut or on NT.
 #include "api.h"
 #include "common.cuh"
@@ -53,12 +53,40 @@ template <> struct Piece<float> {
     }
 };
 
+// The sums of V values over a warp at once: after each of the first log2(V) exchanges a lane goes on with half of the values,
+// so that V = 8 takes 9 shuffles instead of 40.  Every value's sum is formed in the order of warp_sum.  Returns the lane's
+// value; `which` is its number.
+template <int V>
+__device__ __forceinline__ float warp_sums(float (&v)[V], int lane, int& which) {
+    which = 0;
+#pragma unroll
+    for (int o = 16, n = V; o > 0; o >>= 1) {
+        if (n > 1) {
+            n >>= 1;
+            const bool upper = (lane & o) != 0;
+#pragma unroll
+            for (int i = 0; i < V / 2; ++i) {
+                if (i < n) {
+                    const float send = upper ? v[i] : v[i + n], mine = upper ? v[i + n] : v[i];
+                    v[i] = mine + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+            which += upper ? n : 0;
+        } else {
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+        }
+    }
+    return v[0];
+}
+
 // VEC: pieces of 16 bytes (head_dim a whole number of them), else single values.  CPT: pieces a thread owns.  NT: tokens at a
 // time.  TAPS: the most taps this instance takes.  SINGLE: a block per token (a step of single tokens).
 template <typename T, bool VEC, int CPT, int NT, int TAPS, bool SINGLE>
 __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepareArgs a) {
     constexpr int N = VEC ? Piece<T>::N : 1;
     __shared__ float part[2 * NT][32], total[2 * NT];
+    __shared__ long long cache_at[NT];                      // where a token's key and value rows of head 0 lie in the cache
+    __shared__ int cache_row[NT];                           // the row's place in its page; -1: not written
     int seq, r0, past;
     if (SINGLE) {
         const int t = blockIdx.x, pos = a.tok_pos[t];
@@ -104,6 +132,14 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
             f[0] = *p;
         }
     };
+    auto keep_floats = [](float* p, const float (&f)[N]) {
+        if constexpr (VEC) {
+#pragma unroll
+            for (int e = 0; e < N; e += 4) *reinterpret_cast<float4*>(p + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+        } else {
+            *p = f[0];
+        }
+    };
     auto store = [](T* p, const float (&f)[N]) {
         if constexpr (VEC) *reinterpret_cast<uint4*>(p) = Piece<T>::pack(f);
         else *p = from_float<T>(f[0]);
@@ -134,8 +170,18 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
                 for (int e = 0; e < N; ++e) w[k][e] = k == 0 ? 1.f : 0.f;
         }
     };
+    const int end = min(r0 + TAPS, n);
+    // where the cache rows of the tokens from rb on lie
+    auto places = [&](int rb) {
+        if (threadIdx.x >= NT) return;
+        const int p = past + rb + threadIdx.x;
+        // In a ring a later token of this step may land on the same row: only the last writer writes.
+        const bool write = a.do_write && rb + (int)threadIdx.x < end && (long long)p + (long long)a.ring_pages * a.page_size >= (long long)a.seq_end[seq];
+        cache_row[threadIdx.x] = write ? p % a.page_size : -1;
+        cache_at[threadIdx.x] = write ? rdl_cache_offset(a.tables + (long long)seq * a.table_width, p, a.page_size, a.ring_pages, a.n_kv_heads, 0, D) : 0;
+    };
     // What no kernel of this step has written is fetched while the product before this kernel is still running: the model's
-    // constants and, for single tokens, the state (the step before left it, many kernels ago).
+    // constants, the page lists and, for single tokens, the state (the step before left it, many kernels ago).
     constexpr bool EARLY = CPT == 1;
     float bias[N], w[TAPS][N], norm0[N], old[SINGLE && EARLY ? TAPS - 1 : 1][N];
     if (EARLY) {
@@ -151,15 +197,19 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
                         for (int e = 0; e < N; ++e) old[SINGLE ? k - 1 : 0][e] = 0.f;
                 }
             }
-            if (SINGLE && a.wq && c < qw + kw) floats(c < qw ? a.wq + c : a.wk + (c - qw), norm0);
+            if (a.wq && c < qw + kw) floats(c < qw ? a.wq + c : a.wk + (c - qw), norm0);
         }
     }
+    places(r0);
     rdl_grid_wait();
     rdl_grid_launch_dependents();
-    const int end = min(r0 + TAPS, n);
     for (int rb = r0; rb < end; rb += NT) {
         float acc[NT][CPT][N];
         float sums[2 * NT];
+        if (rb != r0) {
+            __syncthreads();                                // what the tokens before left in shared memory is no longer read
+            places(rb);
+        }
 #pragma unroll
         for (int i = 0; i < 2 * NT; ++i) sums[i] = 0.f;
 #pragma unroll
@@ -199,25 +249,33 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
                         sums[2 * i] += c < qw ? s : 0.f;
                         sums[2 * i + 1] += c < qw ? 0.f : s;
                     }
+                } else if (first) {
+                    float f[NT][N];
+#pragma unroll
+                    for (int i = 0; i < NT; ++i)
+                        if (rb + i < end) load(first + (long long)(rb + i) * a.v_first_stride + (c - qw - kw), f[i]);
+#pragma unroll
+                    for (int i = 0; i < NT; ++i)
+#pragma unroll
+                        for (int e = 0; e < N; ++e) acc[i][it][e] = (1.0f - a.v_lambda) * acc[i][it][e] + a.v_lambda * f[i][e];
                 }
             }
         }
         float inv[2 * NT];
         if (a.wq) {
-            __syncthreads();                                // the sums of the tokens before are no longer read
-#pragma unroll
-            for (int i = 0; i < 2 * NT; ++i) {
-                const float s = warp_sum(sums[i]);
-                if (lane == 0) part[i][warp] = s;
-            }
-            __syncthreads();
+            int which;
+            const float s = warp_sums(sums, lane, which);
+            if ((lane & (16 / NT - 1)) == 0) part[which][warp] = s;
+        }
+        __syncthreads();
+        if (a.wq) {
             for (int i = warp; i < 2 * NT; i += n_warps) {
                 const float s = warp_sum(lane < n_warps ? part[i][lane] : 0.f);
-                if (lane == 0) total[i] = s;
+                if (lane == 0) total[i] = 1.0f / sqrtf(s / ((i & 1) ? a.k_count : a.q_count) + a.eps);
             }
             __syncthreads();
 #pragma unroll
-            for (int i = 0; i < 2 * NT; ++i) inv[i] = 1.0f / sqrtf(total[i] / ((i & 1) ? a.k_count : a.q_count) + a.eps);
+            for (int i = 0; i < 2 * NT; ++i) inv[i] = total[i];
         }
 #pragma unroll
         for (int it = 0; it < CPT; ++it) {
@@ -226,7 +284,7 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
             const bool is_q = c < qw, is_k = !is_q && c < qw + kw;
             float wn[N];
             if (a.wq && (is_q || is_k)) {
-                if constexpr (SINGLE && EARLY) {
+                if constexpr (EARLY) {
 #pragma unroll
                     for (int e = 0; e < N; ++e) wn[e] = norm0[e];
                 } else {
@@ -246,20 +304,12 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
 #pragma unroll
                         for (int e = 0; e < N; ++e) v[e] = v[e] * s * wn[e];
                     }
-                } else if (first) {
-                    float f[N];
-                    load(first + (long long)r * a.v_first_stride + (c - qw - kw), f);
-#pragma unroll
-                    for (int e = 0; e < N; ++e) v[e] = (1.0f - a.v_lambda) * v[e] + a.v_lambda * f[e];
                 }
                 store(out + (long long)r * a.out_stride + c, v);
-                if (is_q || !a.do_write) continue;
-                const int p = past + r;
-                // In a ring a later token of this step may land on the same row: only the last writer writes.
-                if ((long long)p + (long long)a.ring_pages * a.page_size < (long long)a.seq_end[seq]) continue;
-                T* dst = (T*)(is_k ? a.k_cache : a.v_cache) +
-                         rdl_cache_offset(a.tables + (long long)seq * a.table_width, p, a.page_size, a.ring_pages, a.n_kv_heads, head, D);
-                const int pr = p % a.page_size;             // chunks of a cache row are stored swizzled by its place in the page
+                const int pr = cache_row[i];
+                if (is_q || pr < 0) continue;
+                // chunks of a cache row are stored swizzled by its place in the page
+                T* dst = (T*)(is_k ? a.k_cache : a.v_cache) + cache_at[i] + (long long)head * a.page_size * D;
                 store(dst + (VEC ? rdl_swizzled_chunk(pr, d / N, D / N) * N : rdl_cache_col<T>(pr, d, D)), v);
             }
         }
@@ -276,11 +326,21 @@ __global__ void __launch_bounds__(VEC ? 512 : 1024) qkv_prepare_kernel(QkvPrepar
                 for (int e = 0; e < N; ++e) bias[e] = 0.f;
                 if (a.bias) floats(a.bias + c, bias);
             }
+            if (SINGLE && EARLY && n == 1) {                // one token moves the state on by one row, and the rows are at hand
+                float u[N];
+                projected(0, c, bias, u);
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k)
+                    if (k < keep) {
+                        if (k == 0) keep_floats(st + (long long)(keep - 1) * C + c, u);
+                        else keep_floats(st + (long long)(keep - 1 - k) * C + c, old[SINGLE && EARLY && k > 0 ? k - 1 : 0]);
+                    }
+                continue;
+            }
             for (int j = 0; j < keep; ++j) {
                 float u[N];
                 projected(n - keep + j, c, bias, u);
-#pragma unroll
-                for (int e = 0; e < N; ++e) st[(long long)j * C + c + e] = u[e];
+                keep_floats(st + (long long)j * C + c, u);
             }
         }
     }

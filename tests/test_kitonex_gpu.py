@@ -159,6 +159,31 @@ def test_bias_convolution_norms_blending_and_cache_write(dtype, sizes):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+def test_preparation_of_many_sequences(dtype):
+    """Forty sequences of 1 to 30 new tokens, some with earlier ones, in one step and each in a step of its own."""
+    from rust_deeplearning_b200.kernels import ops
+    rng = np.random.default_rng(8)
+    H, G, D, taps, n = 3, 1, 16, 4, 40
+    C = (H + 2 * G) * D
+    lens = [int(v) for v in rng.integers(1, 31, size=n)]
+    lens[3:9] = [1] * 6
+    past = [int(v) for v in rng.choice([0, 0, 1, 2, 5, 64], size=n)]
+    slots = [int(v) for v in rng.permutation(n)]
+    rows = _t(rng.normal(size=(sum(lens), C)), dtype)
+    kw = dict(bias=_t(rng.normal(size=C), "float32"), conv=_t(rng.normal(size=(taps, C)), dtype), wq=_t(rng.normal(size=H * D), "float32"),
+              wk=_t(rng.normal(size=G * D), "float32"), eps=1e-5, q_count=H * D, k_count=G * D)
+    before = _t(rng.normal(size=(n, taps - 1, C)), "float32")
+    together, alone = before.clone(), before.clone()
+    got = ops.qkv_prepare(rows, H, G, D, state=together, **kw, **Batch(lens, past, slots).kw())
+    at = 0
+    for i in range(n):
+        one = ops.qkv_prepare(rows[at:at + lens[i]], H, G, D, state=alone, **kw, **Batch([lens[i]], [past[i]], [slots[i]]).kw())
+        assert torch.equal(one, got[at:at + lens[i]]), f"sequence {i}: {lens[i]} tokens after {past[i]}"
+        at += lens[i]
+    assert torch.equal(together, alone)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_preparation_in_a_ring_and_without_its_mechanisms(dtype):
     """With nothing asked for the rows pass through unchanged; in a ring only the last writer of a cache row writes."""
     from rust_deeplearning_b200.kernels import ops
