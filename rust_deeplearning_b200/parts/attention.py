@@ -23,15 +23,15 @@ Optional parameters, for designs that have them (the reference's attention has n
                and the weights are not normalised over the keys
   cache_window the keys the cache keeps per sequence where later runs that read this run's keys look further back than
                this run's own window (default: the window; "all": every key)
-  biases       added to the q, k and v projections (tensor roles "q_bias", "k_bias", "v_bias")
-  conv_taps    a causal convolution over time on every channel of q, k and v, directly after the projections (tensor roles
-               "q_conv", "k_conv", "v_conv", [channels, taps]); the last taps - 1 projected values are state per sequence
+  (biases)     tensor roles "q_bias", "k_bias", "v_bias": added to the projections
+  (convolution)  a causal convolution over time on every channel of q, k and v, directly after the projections (tensor
+               roles "q_conv", "k_conv", "v_conv", [channels, taps]); the last taps - 1 projected values are state per sequence
   chunk        positions form chunks of so many, counted from the sequence's start, and a query sees its own chunk's keys only
                (not together with a window); the cache keeps one chunk's keys
-  distance_bias  {"max": D}: a learned number per head and bucket of distances is added to the scaled scores (tensor role "rel",
-               [buckets, heads]; `distance_buckets`)
+  distance_bias  {"max", "longest"}: a learned number per head and bucket of distances is added to the scaled scores (tensor role "rel",
+               [buckets, heads]; `distance_buckets`; longest: the most positions a query looks back over, itself included)
   off_by_one   one joins the softmax's denominator: a sink whose logit is 0, for every head
-  v_mix        {"name", "first", "lambda"}: v <- (1 - lambda) v + lambda v_first with the values a layer built with first = True
+  v_mix        {"name", "first"}: v <- (1 - lambda) v + lambda v_first with the values a layer built with first = True
                left under that name for this step's tokens (tensor role "v_mix" holds lambda; the mixed values are cached)
 A run that reads another run's keys and values is built without wk and wv.
 With any of them the mixer makes q, k, v and the gate's logits in one product and takes `ops.rope_norm_cache`

@@ -23,7 +23,7 @@ class GatedMLP:
     def __init__(self, hidden_size, intermediate_size, activation, w_gate, w_up, w_down, activation_param=0.0):
         if activation not in ops.GATED_FORMS:
             raise ValueError(f"gated_mlp: unknown activation '{activation}', known: {sorted(ops.GATED_FORMS)}")
-        self.activation_param = float(activation_param)
+        self.form = {"param": float(activation_param)} if activation_param else {}      # of a gated form that has a parameter
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
         self.w_gate_up = torch.cat([w_gate, w_up], dim=0).contiguous()
         self.w_down = w_down
@@ -32,7 +32,7 @@ class GatedMLP:
     delivers_branch = True         # the last product may deliver the result through a stream's sink
 
     def forward(self, x, sink=None):
-        return ops.linear_branch(ops.linear_gated(x, self.w_gate_up, self.activation, param=self.activation_param), self.w_down, sink)
+        return ops.linear_branch(ops.linear_gated(x, self.w_gate_up, self.activation, **self.form), self.w_down, sink)
 
 
 def _build_gated_mlp(spec: PartSpec, ctx: BuildContext) -> GatedMLP:
