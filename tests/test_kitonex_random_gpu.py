@@ -17,7 +17,7 @@ import model_helpers as mh
 import plain_kitonex as plain
 
 pytestmark = pytest.mark.gpu
-MARGIN = {"float32": 2e-5, "bfloat16": 1.2e-2}
+MARGIN = {"float32": 2e-5, "bfloat16": 2.5e-2}
 
 
 def _mlp(rng):
