@@ -11,7 +11,7 @@ extern "C" {
 #define RDL_ACT_SILU 1
 #define RDL_ACT_SWISH_LIMIT 2   // min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1), L a parameter
 
-#define RDL_ABI_VERSION 20
+#define RDL_ABI_VERSION 21
 
 const char* rdl_last_error(void);
 int rdl_abi_version(void);
@@ -78,6 +78,9 @@ typedef struct {
     // entry stands for every larger distance); NULL: none.  rdl_attention_plain takes it as it is, the bfloat16 kernels
     // (prefill, prefill_tc, decode) take it times log2(e)
     const float* rel_bias; int rel_len;
+    // decode kernel, optional: kv_share > 1 - so many consecutive of the n_kv_heads read the same key/value head of the cache
+    // (a group of query heads too large for one block, cut into kv_share equal ones); not together with new_rows
+    int kv_share;
     // filled in by the launcher: clock cycles after which a wait is given up, and the test's extra bytes
     long long wait_cycles; int test_extra_tx;
 } AttentionArgs;
@@ -95,8 +98,11 @@ long long rdl_attention_decode_scratch_bytes(int n_tokens, int n_heads, int n_kv
 int rdl_embed_rows(void* out_f32, const void* table, int table_dtype, const int* ids, float scale,
                    int n_rows, int hidden, int vocab, int* status, const void* pos_table, int pos_dtype,
                    const int* tok_pos, int n_pos, void* stream);
+// t = norm1(x) or x;  h = res + t (or t) + add_rows[row] + add_vec;  res_out <- h;  y <- norm2(h) or h.
+// res, res_out (may be the same buffer), add_rows (float [rows][hidden]), add_vec (float [hidden]), the norms and y are optional.
 int rdl_norm_residual_norm(const void* x, int x_dtype, const int* row_index,
-                           const void* w1, int w1_dtype, float eps1, float off1, void* res_f32,
+                           const void* w1, int w1_dtype, float eps1, float off1, const void* res_f32, void* res_out_f32,
+                           const float* add_rows, const float* add_vec,
                            const void* w2, int w2_dtype, float eps2, float off2,
                            void* y, int y_dtype, int n_rows, int hidden, void* stream);
 int rdl_gated_activation(void* out, const void* gate_up, int dtype, int activation, int n_rows, int inter, float act_param, void* stream);
@@ -219,6 +225,71 @@ int rdl_gated_residual_add(float* res, const void* gates, long long gates_stride
 #define RDL_UNARY_RELU2 16     // max(x, 0)^2
 #define RDL_UNARY_SILU 17
 int rdl_activation_inplace(void* x, int dtype, long long total, int act, void* stream);
+
+// ---- what lies between a q/k/v product and attention, head by head (csrc/head_prepare.cu) ----
+// bias, short causal convolution, values (columns of their own or the keys as the convolution left them), a norm per head,
+// rotation, a factor on the queries by position, the laying out of heads with several maps, and the cache write; every
+// mechanism but the last two optional.
+typedef struct {
+    int dtype;
+    int n_tokens, n_seqs;
+    int n_heads, n_kv_heads, maps;             // every query and key head has `maps` maps
+    int dim, vdim, pad;                        // values of a map, of a value head, and of a head in `out` and in the cache
+    const void* rows; long long row_stride;
+    int q_col, k_col, v_col;                   // heads lie map by map from each column; v_col < 0: the keys serve as values
+    void* out; long long out_stride;           // [n_heads * maps][pad] queries, then [n_kv_heads][pad] keys and as many values
+    const float* bias;                         // [channels] of q and k
+    const void* conv; int taps; float* state;  // [taps][channels] in dtype; float [slots][taps - 1][channels]
+    const float* wq; const float* wk; float eps;           // [dim] each
+    const float* cos_t; const float* sin_t; int rot_n;     // [positions][rot_n / 2]
+    const float* q_factor;                     // [positions]
+    const int* tok_pos; const int* seq_start; const int* slots; const int* seq_end;
+    int write_kv;                              // 1: keys and values also go to `out` (0: only to the cache)
+    int do_write;
+    void* k_cache; void* v_cache; const int* tables; int table_width, page_size, ring_pages;
+} HeadPrepareArgs;
+int rdl_head_prepare(const HeadPrepareArgs* a, void* stream);
+
+// ---- attention or recurrence results made into the output product's rows (csrc/context_finish.cu) ----
+#define RDL_CONTEXT_GATE_NONE 0
+#define RDL_CONTEXT_GATE_HEAD 1      // one number per head
+#define RDL_CONTEXT_GATE_VALUE 2     // one per value
+typedef struct {
+    const void* x; int x_f32; long long x_stride; int x_head;    // head h, map m at column (h * maps + m) * x_head; float or dtype
+    int n_heads, vdim;
+    int maps; float lambda;                    // 2: x_1 - lambda x_2
+    int norm; float eps;                       // 1: divided by its root mean square
+    const float* weight;                       // optional [n_heads * vdim]
+    float factor;
+    const void* gate; long long gate_stride; int gate_kind;      // in dtype
+    int out_col;
+} ContextSide;
+typedef struct {
+    int dtype, n_tokens, n_sides;
+    ContextSide side[2];
+    void* out; long long out_stride; int out_width;
+    int ones_col, n_ones;                      // columns from ones_col on: n_ones ones, then zeros up to out_width
+} ContextFinishArgs;
+int rdl_context_finish(const ContextFinishArgs* a, void* stream);
+
+// ---- the matrix memory of xLSTM (csrc/matrix_memory.cu, csrc/matrix_memory_chunked.cu) ----
+typedef struct {
+    int dtype;                                  // of the packed rows
+    int n_tokens, n_seqs, n_heads, dim, vdim;
+    const void* rows; long long row_stride;
+    int q_col, k_col, v_col, i_col, f_col;      // heads one after another; a gate logit per head
+    const float* i_bias; const float* f_bias;   // [heads]
+    float cap, q_scale, den_eps;
+    const int* tok_pos; const int* seq_start; const int* slots;
+    float* state;                               // [slots][heads][dim][vdim]
+    float* norm;                                // [slots][heads][rdl_matrix_memory_copies(vdim)][dim + 1]: n, then m times log2(e)
+    float* out;                                 // [tokens][heads * vdim]
+} MatrixMemoryArgs;
+int rdl_matrix_memory_scan(const MatrixMemoryArgs* a, void* stream);
+int rdl_matrix_memory_copies(int vdim);
+// bfloat16 rows, sizes in multiples of 16 (dim up to 128), q, k and v on 16-byte boundaries; three launches
+int rdl_matrix_memory_chunked(const MatrixMemoryArgs* a, void* work, long long work_bytes, void* stream);
+long long rdl_matrix_memory_chunked_work_bytes(int n_tokens, int n_seqs, int n_heads, int dim, int vdim);
 
 // ---- recurrences whose decay depends on the token (csrc/recurrence.cu) ----
 #define RDL_REC_SSM 0

@@ -119,6 +119,8 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     const int t = blockIdx.z, g = blockIdx.y, sp = blockIdx.x;
     const int hd = EXACT ? HD : a.head_dim, ps = a.page_size;
     const int G = a.n_heads / a.n_kv_heads;
+    // the cache's key/value heads, and this block's (several blocks' groups of query heads may share one)
+    const int share = a.kv_share > 1 ? a.kv_share : 1, cache_heads = a.n_kv_heads / share, cg = g / share;
     // The page list can only be read once the token's sequence and position are known: two trips to memory one
     // after the other, at a time when the kernel before this one keeps the memory system busy.  In a decode
     // step token t usually is sequence t and a run that does not start inside a window begins at page
@@ -156,7 +158,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
     // lands too), so this runs while the earlier kernel is still finishing.
     if (tid <= page_last - page_first) {
         const int page = table[(page_first + tid) % a.ring_pages];
-        const long long off = ((long long)page * a.n_kv_heads + g) * ps * hd;
+        const long long off = ((long long)page * cache_heads + cg) * ps * hd;
         asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(kcache + off), "r"(ps * row_bytes) : "memory");
         asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(vcache + off), "r"(ps * row_bytes) : "memory");
     }
@@ -179,7 +181,7 @@ __global__ void __launch_bounds__(DEC_THREADS) attention_decode_kernel(Attention
         if (*gave_up) return;
         issued = i + 1;
         const int page = table[(page_first + (i >> 1)) % a.ring_pages];
-        const long long off = ((long long)page * a.n_kv_heads + g) * ps * hd;
+        const long long off = ((long long)page * cache_heads + cg) * ps * hd;
         const uint32_t place = (uint32_t)(i % 3);
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
         mbar_expect_tx(bars + 8 * place, tile_bytes + (i == 0 ? (uint32_t)a.test_extra_tx : 0u));
@@ -642,6 +644,8 @@ extern "C" int rdl_attention_decode(const AttentionArgs* a, void* stream) {
     const int G = a->n_heads / a->n_kv_heads;
     RDL_REQUIRE(G <= QROWS, "attention_decode: %d query heads per key/value head, at most %d are supported", G, QROWS);
     RDL_REQUIRE(a->tables && a->k_cache && a->v_cache, "attention_decode: needs a cache");
+    RDL_REQUIRE(a->kv_share >= 0 && (a->kv_share <= 1 || (a->n_kv_heads % a->kv_share == 0 && !a->new_rows)),
+                "attention_decode: %d key/value heads cannot share in groups of %d (or the step's rows are not written yet)", a->n_kv_heads, a->kv_share);
     RDL_REQUIRE(a->page_size % 16 == 0 && a->page_size <= 16 * DEC_WARPS,
                 "attention_decode: page_size %d must be a multiple of 16 and at most %d", a->page_size, 16 * DEC_WARPS);
     RDL_REQUIRE(a->keys_per_split > 0 && a->keys_per_split % a->page_size == 0,

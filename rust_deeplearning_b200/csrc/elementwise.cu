@@ -61,7 +61,7 @@ extern "C" int rdl_embed_rows(void* out_f32, const void* table, int table_dtype,
 // ---------------------------------------------------------------------------------------------
 // fused norm / residual / norm
 //   t = w1 ? rms_norm(x; w1, eps1, off1) : x
-//   h = res ? res + t : t ;  res <- h (float) when res is given
+//   h = (res ? res + t : t) + add_rows[r] + add_vec (each optional) ;  res_out <- h (float) when given
 //   y = w2 ? rms_norm(h; w2, eps2, off2) : h          (written when y is given)
 // x rows may be gathered through row_index.
 // ---------------------------------------------------------------------------------------------
@@ -69,7 +69,8 @@ struct NormArgs {
     const void* x; int x_dtype;
     const int* row_index;
     const void* w1; int w1_dtype; float eps1, off1;
-    float* res;
+    const float* res; float* res_out;
+    const float* add_rows; const float* add_vec;
     const void* w2; int w2_dtype; float eps2, off2;
     void* y; int y_dtype;
     int hidden;
@@ -97,10 +98,12 @@ __global__ void norm_residual_norm_kernel(NormArgs a) {
         for (int j = threadIdx.x; j < H; j += blockDim.x)
             row[j] = row[j] * inv * (rdl_load(a.w1, j, a.w1_dtype) + a.off1);
     }
-    if (a.res) {
+    if (a.res || a.res_out || a.add_rows || a.add_vec) {
         for (int j = threadIdx.x; j < H; j += blockDim.x) {
-            const float h = a.res[out + j] + row[j];
-            a.res[out + j] = h;
+            float h = a.res ? a.res[out + j] + row[j] : row[j];
+            if (a.add_rows) h += a.add_rows[out + j];
+            if (a.add_vec) h += a.add_vec[j];
+            if (a.res_out) a.res_out[out + j] = h;
             row[j] = h;
         }
     }
@@ -197,10 +200,24 @@ __global__ void __launch_bounds__(THREADS, norm_min_blocks(ITER, THREADS, LATE))
     }
     if (a.res) {
 #pragma unroll
+        for (int i = 0; i < ITER; ++i) { xv[i].x += rv[i].x; xv[i].y += rv[i].y; xv[i].z += rv[i].z; xv[i].w += rv[i].w; }
+    }
+    if (a.add_rows || a.add_vec) {           // rows and a vector that join the stream here (a loop's entry)
+#pragma unroll
         for (int i = 0; i < ITER; ++i) {
             const int j = (i * THREADS + threadIdx.x) * 4;
-            xv[i].x += rv[i].x; xv[i].y += rv[i].y; xv[i].z += rv[i].z; xv[i].w += rv[i].w;
-            if (j < H) *reinterpret_cast<float4*>(a.res + out + j) = xv[i];
+            if (j >= H) continue;
+            const float4 r4 = a.add_rows ? *reinterpret_cast<const float4*>(a.add_rows + out + j) : zero;
+            const float4 v4 = a.add_vec ? *reinterpret_cast<const float4*>(a.add_vec + j) : zero;
+            xv[i].x = xv[i].x + r4.x + v4.x; xv[i].y = xv[i].y + r4.y + v4.y;
+            xv[i].z = xv[i].z + r4.z + v4.z; xv[i].w = xv[i].w + r4.w + v4.w;
+        }
+    }
+    if (a.res_out) {
+#pragma unroll
+        for (int i = 0; i < ITER; ++i) {
+            const int j = (i * THREADS + threadIdx.x) * 4;
+            if (j < H) *reinterpret_cast<float4*>(a.res_out + out + j) = xv[i];
         }
     }
     if (!a.y) return;
@@ -232,13 +249,13 @@ static bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
 extern "C" int rdl_norm_residual_norm(const void* x, int x_dtype, const int* row_index,
                                       const void* w1, int w1_dtype, float eps1, float off1,
-                                      void* res_f32,
+                                      const void* res_f32, void* res_out_f32, const float* add_rows, const float* add_vec,
                                       const void* w2, int w2_dtype, float eps2, float off2,
                                       void* y, int y_dtype, int n_rows, int hidden, void* stream) {
     if (hidden > 0 && hidden % 4 == 0 && hidden <= 8192 && n_rows > 0 && rdl_valid_dtype(x_dtype) && rdl_valid_dtype(y_dtype) &&
-        (!w1 || rdl_valid_dtype(w1_dtype)) && (!w2 || rdl_valid_dtype(w2_dtype)) && !(row_index && res_f32) && (y || res_f32) &&
-        aligned16(x) && aligned16(res_f32) && aligned16(w1) && aligned16(w2) && aligned16(y)) {
-        NormArgs a{x, x_dtype, row_index, w1, w1_dtype, eps1, off1, (float*)res_f32, w2, w2_dtype, eps2, off2, y, y_dtype, hidden};
+        (!w1 || rdl_valid_dtype(w1_dtype)) && (!w2 || rdl_valid_dtype(w2_dtype)) && !(row_index && (res_f32 || res_out_f32 || add_rows)) && (y || res_out_f32) &&
+        aligned16(x) && aligned16(res_f32) && aligned16(res_out_f32) && aligned16(add_rows) && aligned16(add_vec) && aligned16(w1) && aligned16(w2) && aligned16(y)) {
+        NormArgs a{x, x_dtype, row_index, w1, w1_dtype, eps1, off1, (const float*)res_f32, (float*)res_out_f32, add_rows, add_vec, w2, w2_dtype, eps2, off2, y, y_dtype, hidden};
         cudaStream_t st = (cudaStream_t)stream;
         cudaError_t e;
         // Threads per row: few rows (decode) want the row spread over many threads; many rows (prefill) want
@@ -279,8 +296,8 @@ extern "C" int rdl_norm_residual_norm(const void* x, int x_dtype, const int* row
     RDL_REQUIRE(!w1 || rdl_valid_dtype(w1_dtype), "norm: bad dtype of the first weight");
     RDL_REQUIRE(!w2 || rdl_valid_dtype(w2_dtype), "norm: bad dtype of the second weight");
     RDL_REQUIRE(n_rows >= 0 && hidden > 0, "norm: bad sizes rows=%d hidden=%d", n_rows, hidden);
-    RDL_REQUIRE(!(row_index && res_f32), "norm: gathered rows cannot be combined with a residual");
-    RDL_REQUIRE(y || res_f32, "norm: nothing to write");
+    RDL_REQUIRE(!(row_index && (res_f32 || res_out_f32 || add_rows)), "norm: gathered rows cannot be combined with a residual");
+    RDL_REQUIRE(y || res_out_f32, "norm: nothing to write");
     const size_t smem = (size_t)hidden * sizeof(float);
     RDL_REQUIRE(smem <= 200 * 1024, "norm: hidden size %d needs %zu bytes of shared memory, limit is 204800", hidden, smem);
     if (n_rows == 0) return 0;
@@ -291,7 +308,7 @@ extern "C" int rdl_norm_residual_norm(const void* x, int x_dtype, const int* row
             granted = smem;
         }
     }
-    NormArgs a{x, x_dtype, row_index, w1, w1_dtype, eps1, off1, (float*)res_f32, w2, w2_dtype, eps2, off2, y, y_dtype, hidden};
+    NormArgs a{x, x_dtype, row_index, w1, w1_dtype, eps1, off1, (const float*)res_f32, (float*)res_out_f32, add_rows, add_vec, w2, w2_dtype, eps2, off2, y, y_dtype, hidden};
     const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
     RDL_CHECK_EX(rdl_launch(norm_residual_norm_kernel, dim3(n_rows), dim3(threads), smem, (cudaStream_t)stream, a), "norm_residual_norm");
     return 0;

@@ -391,6 +391,7 @@ __global__ void __launch_bounds__(ST_THREADS, 2) gemm_stream_kernel(const __grid
                     }
                     float y = sc.y * (h0 + sc.x * a0);
                     if (GATED) y = rdl_gated(y, sc.y * (h1 + sc.x * a1), a.activation, a.act_param);
+                    else if (a.activation >= 16) y = rdl_unary(y, a.activation);
                     if (a.softcap > 0.f) y = a.softcap * tanhf(y / a.softcap);
                     rdl_store(a.out, (long long)j * a.N + n, a.out_dtype, y);
                 }

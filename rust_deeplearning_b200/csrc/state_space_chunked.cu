@@ -17,68 +17,16 @@
 // tensor-core product - the weighted x of step 1, P, and the state S - goes in as two bfloat16 terms (its rounding and
 // what the rounding left), so that 16 bits of it count; every sum is float.  dt, the decays and their logarithms are float.
 #include "api.h"
+#include "chunk_mma.cuh"
 #include "common.cuh"
 #include "launch.cuh"
 
 namespace {
 
-#define SSC_CHUNK 64
 #define SSC_COLS 64
 #define SSC_THREADS 256
-#define SSC_PAD 8            // bfloat16 values between rows in shared memory: ldmatrix reads eight rows without bank conflicts
 
-__device__ __forceinline__ uint32_t ssc_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void ssc_ldm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ssc_ldm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ssc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t ssc_pack(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&v);
-}
-// a pair of floats as two bfloat16 pairs: the rounding, and what it left
-__device__ __forceinline__ void ssc_split(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const float2 f = __bfloat1622float2(h);
-    hi = *reinterpret_cast<const uint32_t*>(&h);
-    lo = ssc_pack(x - f.x, y - f.y);
-}
 __device__ __forceinline__ float ssc_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-
-// chunks a step can have at most (every sequence may end in a partial chunk)
-static inline int ssc_max_chunks(int n_tokens, int n_seqs) {
-    const int by_tokens = n_tokens / SSC_CHUNK + n_seqs;
-    return by_tokens < n_tokens ? by_tokens : n_tokens;
-}
-
-// chunk number `idx` of the step -> its sequence and its first token there; false beyond the step's last chunk
-__device__ __forceinline__ bool ssc_find_chunk(const RecurrenceArgs& a, int idx, int& seq, int& t0) {
-    for (int s = 0; s < a.n_seqs; ++s) {
-        const int n = a.seq_start[s + 1] - a.seq_start[s];
-        const int nc = (n > 0 && a.tok_pos[a.seq_start[s]] >= 0) ? (n + SSC_CHUNK - 1) / SSC_CHUNK : 0;
-        if (idx < nc) { seq = s; t0 = idx * SSC_CHUNK; return true; }
-        idx -= nc;
-    }
-    return false;
-}
-
-// 64 rows of `width` bfloat16 values (a multiple of 8) from packed rows into shared memory, 16 bytes a copy; rows from L on are zeros
-__device__ __forceinline__ void ssc_fill(__nv_bfloat16* dst, int dst_stride, const __nv_bfloat16* src, long long src_stride, int width, int L, int tid) {
-    const int per = width >> 3;
-    for (int idx = tid; idx < SSC_CHUNK * per; idx += SSC_THREADS) {
-        const int j = idx / per, c = (idx - j * per) << 3;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (j < L) v = *reinterpret_cast<const uint4*>(src + (long long)j * src_stride + c);
-        *reinterpret_cast<uint4*>(dst + j * dst_stride + c) = v;
-    }
-}
 
 template <bool OUTPUT>
 __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a, float* __restrict__ totals, float* __restrict__ work) {
@@ -86,20 +34,20 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
     const int dim = a.dim, vdim = a.vdim;
     const int h = blockIdx.y, c0 = blockIdx.z * SSC_COLS;
     const int nv = min(SSC_COLS, vdim - c0);               // columns of this block (a multiple of 16)
-    const int qs = dim + SSC_PAD, vs = SSC_COLS + SSC_PAD;  // row strides in shared memory, in values
+    const int qs = dim + CM_PAD, vs = SSC_COLS + CM_PAD;  // row strides in shared memory, in values
     __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(ssc_raw);    // [64][qs]  B
-    __nv_bfloat16* Vh = Ks + SSC_CHUNK * qs;                            // [64][vs]  x (OUTPUT), or the weighted x's rounding
-    __nv_bfloat16* Vl = Vh + SSC_CHUNK * vs;                            // [64][vs]  what that rounding left (not OUTPUT)
-    __nv_bfloat16* Qs = Vl + SSC_CHUNK * vs;                            // [64][qs]  C        OUTPUT only, like the two below
-    __nv_bfloat16* Sh = Qs + SSC_CHUNK * qs;                            // [dim][vs] the state before the chunk, rounded
+    __nv_bfloat16* Vh = Ks + CM_CHUNK * qs;                            // [64][vs]  x (OUTPUT), or the weighted x's rounding
+    __nv_bfloat16* Vl = Vh + CM_CHUNK * vs;                            // [64][vs]  what that rounding left (not OUTPUT)
+    __nv_bfloat16* Qs = Vl + CM_CHUNK * vs;                            // [64][qs]  C        OUTPUT only, like the two below
+    __nv_bfloat16* Sh = Qs + CM_CHUNK * qs;                            // [dim][vs] the state before the chunk, rounded
     __nv_bfloat16* Sl = Sh + dim * vs;                                  // [dim][vs] what the rounding left
-    __shared__ float dts[SSC_CHUNK], cl[SSC_CHUNK];                     // dt_j and c_j
+    __shared__ float dts[CM_CHUNK], cl[CM_CHUNK];                     // dt_j and c_j
     rdl_grid_wait();
     rdl_grid_launch_dependents();
     int seq, t0;
-    if (!ssc_find_chunk(a, blockIdx.x, seq, t0)) return;
+    if (!cm_find_chunk(a.seq_start, a.tok_pos, a.n_seqs, blockIdx.x, seq, t0)) return;
     const int row0 = a.seq_start[seq], n = a.seq_start[seq + 1] - row0;
-    const int L = min(SSC_CHUNK, n - t0);
+    const int L = min(CM_CHUNK, n - t0);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
     const int kh = h / (a.n_heads / a.n_key_heads);
     const int ksteps = dim >> 4, n_mt = dim >> 4, nt_count = nv >> 3;
@@ -123,18 +71,18 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
         dts[j0] = d0; dts[j1] = d1;
         cl[j0] = run - l1; cl[j1] = run;
     }
-    ssc_fill(Ks, qs, rows + a.k_col + kh * dim, a.row_stride, dim, L, tid);
+    cm_fill(Ks, qs, rows + a.k_col + kh * dim, a.row_stride, dim, L, tid, SSC_THREADS);
     if (OUTPUT) {
-        ssc_fill(Qs, qs, rows + a.q_col + kh * dim, a.row_stride, dim, L, tid);
-        ssc_fill(Vh, vs, rows + a.v_col + h * vdim + c0, a.row_stride, nv, L, tid);
+        cm_fill(Qs, qs, rows + a.q_col + kh * dim, a.row_stride, dim, L, tid, SSC_THREADS);
+        cm_fill(Vh, vs, rows + a.v_col + h * vdim + c0, a.row_stride, nv, L, tid, SSC_THREADS);
         // the state before this chunk as two bfloat16 terms
 #pragma unroll 4
         for (int idx = tid; idx < dim * (nv >> 2); idx += SSC_THREADS) {
             const int r = idx / (nv >> 2), c = 4 * (idx - r * (nv >> 2));
             const float4 sv = __ldcg(reinterpret_cast<const float4*>(W + (long long)r * vdim + c));
             uint2 hi, lo;
-            ssc_split(sv.x, sv.y, hi.x, lo.x);
-            ssc_split(sv.z, sv.w, hi.y, lo.y);
+            cm_split(sv.x, sv.y, hi.x, lo.x);
+            cm_split(sv.z, sv.w, hi.y, lo.y);
             *reinterpret_cast<uint2*>(Sh + r * vs + c) = hi;
             *reinterpret_cast<uint2*>(Sl + r * vs + c) = lo;
         }
@@ -144,13 +92,13 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
     if (!OUTPUT) {
         // x_j dt_j 2^(c_(L-1) - c_j), as two terms
         const float c_end = cl[L - 1];
-        for (int idx = tid; idx < SSC_CHUNK * (nv >> 1); idx += SSC_THREADS) {
+        for (int idx = tid; idx < CM_CHUNK * (nv >> 1); idx += SSC_THREADS) {
             const int j = idx / (nv >> 1), c = 2 * (idx - j * (nv >> 1));
             uint32_t hi = 0u, lo = 0u;
             if (j < L) {
                 const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(rows + (long long)j * a.row_stride + a.v_col + h * vdim + c0 + c));
                 const float wj = dts[j] * exp2f(c_end - cl[j]);
-                ssc_split(v.x * wj, v.y * wj, hi, lo);
+                cm_split(v.x * wj, v.y * wj, hi, lo);
             }
             *reinterpret_cast<uint32_t*>(Vh + j * vs + c) = hi;
             *reinterpret_cast<uint32_t*>(Vl + j * vs + c) = lo;
@@ -166,18 +114,18 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
 #pragma unroll
             for (int kb = 0; kb < 4; ++kb) {
                 uint32_t ka[4];
-                ssc_ldm4t(ka, ssc_smem(Ks + (kb * 16 + ((lane >> 4) << 3) + (lane & 7)) * qs + m0 + (((lane >> 3) & 1) << 3)));
+                cm_ldm4t(ka, cm_smem(Ks + (kb * 16 + ((lane >> 4) << 3) + (lane & 7)) * qs + m0 + (((lane >> 3) & 1) << 3)));
 #pragma unroll
                 for (int nb = 0; nb < 4; ++nb) {
                     if (2 * nb >= nt_count) continue;
                     const int off = (kb * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * vs + nb * 16 + ((lane >> 4) << 3);
                     uint32_t bh[4], bl[4];
-                    ssc_ldm4t(bh, ssc_smem(Vh + off));
-                    ssc_ldm4t(bl, ssc_smem(Vl + off));
-                    ssc_mma(u[2 * nb], ka, bh[0], bh[1]);
-                    ssc_mma(u[2 * nb + 1], ka, bh[2], bh[3]);
-                    ssc_mma(u[2 * nb], ka, bl[0], bl[1]);
-                    ssc_mma(u[2 * nb + 1], ka, bl[2], bl[3]);
+                    cm_ldm4t(bh, cm_smem(Vh + off));
+                    cm_ldm4t(bl, cm_smem(Vl + off));
+                    cm_mma(u[2 * nb], ka, bh[0], bh[1]);
+                    cm_mma(u[2 * nb + 1], ka, bh[2], bh[3]);
+                    cm_mma(u[2 * nb], ka, bl[0], bl[1]);
+                    cm_mma(u[2 * nb + 1], ka, bl[2], bl[3]);
                 }
             }
 #pragma unroll
@@ -198,7 +146,7 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
     uint32_t qf[8][4];
 #pragma unroll
     for (int kk = 0; kk < 8; ++kk)
-        if (kk < ksteps) ssc_ldm4(qf[kk], ssc_smem(Qs + (rw * 16 + (lane & 15)) * qs + kk * 16 + 8 * (lane >> 4)));
+        if (kk < ksteps) cm_ldm4(qf[kk], cm_smem(Qs + (rw * 16 + (lane & 15)) * qs + kk * 16 + 8 * (lane >> 4)));
     float p[8][4];
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) p[nt][0] = p[nt][1] = p[nt][2] = p[nt][3] = 0.f;
@@ -209,9 +157,9 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
         for (int kk = 0; kk < 8; ++kk) {
             if (kk >= ksteps) continue;
             uint32_t bf[4];
-            ssc_ldm4(bf, ssc_smem(Ks + (np * 16 + ((lane >> 4) << 3) + (lane & 7)) * qs + kk * 16 + (((lane >> 3) & 1) << 3)));
-            ssc_mma(p[2 * np], qf[kk], bf[0], bf[1]);
-            ssc_mma(p[2 * np + 1], qf[kk], bf[2], bf[3]);
+            cm_ldm4(bf, cm_smem(Ks + (np * 16 + ((lane >> 4) << 3) + (lane & 7)) * qs + kk * 16 + (((lane >> 3) & 1) << 3)));
+            cm_mma(p[2 * np], qf[kk], bf[0], bf[1]);
+            cm_mma(p[2 * np + 1], qf[kk], bf[2], bf[3]);
         }
     }
     const float ci_lo = cl[i_hi - 8], ci_hi = cl[i_hi];
@@ -231,20 +179,20 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
     for (int kb = 0; kb < 4; ++kb) {
         if (kb > rw) continue;
         uint32_t pa[4], pb[4];
-        ssc_split(p[2 * kb][0], p[2 * kb][1], pa[0], pb[0]);
-        ssc_split(p[2 * kb][2], p[2 * kb][3], pa[1], pb[1]);
-        ssc_split(p[2 * kb + 1][0], p[2 * kb + 1][1], pa[2], pb[2]);
-        ssc_split(p[2 * kb + 1][2], p[2 * kb + 1][3], pa[3], pb[3]);
+        cm_split(p[2 * kb][0], p[2 * kb][1], pa[0], pb[0]);
+        cm_split(p[2 * kb][2], p[2 * kb][3], pa[1], pb[1]);
+        cm_split(p[2 * kb + 1][0], p[2 * kb + 1][1], pa[2], pb[2]);
+        cm_split(p[2 * kb + 1][2], p[2 * kb + 1][3], pa[3], pb[3]);
 #pragma unroll
         for (int nl = 0; nl < 2; ++nl) {
             const int nb = 2 * cw + nl;
             if (2 * nb >= nt_count) continue;
             uint32_t bf[4];
-            ssc_ldm4t(bf, ssc_smem(Vh + (kb * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * vs + nb * 16 + ((lane >> 4) << 3)));
-            ssc_mma(o[2 * nl], pa, bf[0], bf[1]);
-            ssc_mma(o[2 * nl + 1], pa, bf[2], bf[3]);
-            ssc_mma(o[2 * nl], pb, bf[0], bf[1]);
-            ssc_mma(o[2 * nl + 1], pb, bf[2], bf[3]);
+            cm_ldm4t(bf, cm_smem(Vh + (kb * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * vs + nb * 16 + ((lane >> 4) << 3)));
+            cm_mma(o[2 * nl], pa, bf[0], bf[1]);
+            cm_mma(o[2 * nl + 1], pa, bf[2], bf[3]);
+            cm_mma(o[2 * nl], pb, bf[0], bf[1]);
+            cm_mma(o[2 * nl + 1], pb, bf[2], bf[3]);
         }
     }
 #pragma unroll
@@ -256,12 +204,12 @@ __global__ void __launch_bounds__(SSC_THREADS) ssc_chunk_kernel(RecurrenceArgs a
             if (2 * nb >= nt_count) continue;
             const int off = (kk * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * vs + nb * 16 + ((lane >> 4) << 3);
             uint32_t bh[4], bl[4];
-            ssc_ldm4t(bh, ssc_smem(Sh + off));
-            ssc_ldm4t(bl, ssc_smem(Sl + off));
-            ssc_mma(o2[2 * nl], qf[kk], bh[0], bh[1]);
-            ssc_mma(o2[2 * nl + 1], qf[kk], bh[2], bh[3]);
-            ssc_mma(o2[2 * nl], qf[kk], bl[0], bl[1]);
-            ssc_mma(o2[2 * nl + 1], qf[kk], bl[2], bl[3]);
+            cm_ldm4t(bh, cm_smem(Sh + off));
+            cm_ldm4t(bl, cm_smem(Sl + off));
+            cm_mma(o2[2 * nl], qf[kk], bh[0], bh[1]);
+            cm_mma(o2[2 * nl + 1], qf[kk], bh[2], bh[3]);
+            cm_mma(o2[2 * nl], qf[kk], bl[0], bl[1]);
+            cm_mma(o2[2 * nl + 1], qf[kk], bl[2], bl[3]);
         }
     }
     const float w_lo = exp2f(ci_lo), w_hi = exp2f(ci_hi);
@@ -294,14 +242,14 @@ __global__ void __launch_bounds__(128) ssc_scan_kernel(RecurrenceArgs a, const f
     int first = 0;                                  // the step's chunks before this sequence's
     for (int s = 0; s < seq; ++s) {
         const int m = a.seq_start[s + 1] - a.seq_start[s];
-        if (m > 0 && a.tok_pos[a.seq_start[s]] >= 0) first += (m + SSC_CHUNK - 1) / SSC_CHUNK;
+        if (m > 0 && a.tok_pos[a.seq_start[s]] >= 0) first += (m + CM_CHUNK - 1) / CM_CHUNK;
     }
     const long long per = (long long)a.dim * a.vdim;          // a multiple of 4 (both sizes are multiples of 16)
     const long long e = 4 * ((long long)blockIdx.z * blockDim.x + threadIdx.x);
     if (e >= per) return;
     float4* S = reinterpret_cast<float4*>(a.state + ((long long)a.slots[seq] * a.n_heads + h) * per + e);
     float4 s = *S;
-    const int chunks = (n + SSC_CHUNK - 1) / SSC_CHUNK;
+    const int chunks = (n + CM_CHUNK - 1) / CM_CHUNK;
     float4* w = reinterpret_cast<float4*>(work + ((long long)first * a.n_heads + h) * per + e);
     const float* tot = totals + (long long)first * a.n_heads + h;
     const long long step = (long long)a.n_heads * per / 4;
@@ -337,7 +285,7 @@ __global__ void __launch_bounds__(128) ssc_scan_kernel(RecurrenceArgs a, const f
 
 // Bytes of the work buffer: the chunks' decays [chunks][heads] (padded to 16 bytes) and a state per chunk and head.
 extern "C" long long rdl_state_space_chunked_work_bytes(int n_tokens, int n_seqs, int n_heads, int dim, int vdim) {
-    const long long chunks = ssc_max_chunks(n_tokens, n_seqs);
+    const long long chunks = cm_max_chunks(n_tokens, n_seqs);
     const long long totals = (chunks * n_heads + 3) / 4 * 4;
     return (totals + chunks * n_heads * dim * vdim) * (long long)sizeof(float);
 }
@@ -355,15 +303,15 @@ extern "C" int rdl_state_space_chunked(const RecurrenceArgs* a, void* work, long
     RDL_REQUIRE(((uintptr_t)a->out & 7) == 0 && ((uintptr_t)a->state & 15) == 0 && ((uintptr_t)work & 15) == 0,
                 "state_space_chunked: the output must be 8-byte aligned, state and work buffer 16-byte aligned");
     if (a->n_tokens == 0 || a->n_seqs == 0) return 0;
-    const int max_chunks = ssc_max_chunks(a->n_tokens, a->n_seqs);
+    const int max_chunks = cm_max_chunks(a->n_tokens, a->n_seqs);
     RDL_REQUIRE(work && work_bytes >= rdl_state_space_chunked_work_bytes(a->n_tokens, a->n_seqs, a->n_heads, a->dim, a->vdim),
                 "state_space_chunked: the work buffer is too small");
     RDL_REQUIRE(a->n_heads <= 65535 && (a->vdim + SSC_COLS - 1) / SSC_COLS <= 65535, "state_space_chunked: too many heads or columns for one grid");
     float* totals = (float*)work;
     float* states = totals + ((long long)max_chunks * a->n_heads + 3) / 4 * 4;
-    const int qs = a->dim + SSC_PAD, vs = SSC_COLS + SSC_PAD;
-    const size_t smem_u = (size_t)(SSC_CHUNK * qs + 2 * SSC_CHUNK * vs) * 2;
-    const size_t smem_o = (size_t)(2 * SSC_CHUNK * qs + 2 * SSC_CHUNK * vs + 2 * a->dim * vs) * 2;
+    const int qs = a->dim + CM_PAD, vs = SSC_COLS + CM_PAD;
+    const size_t smem_u = (size_t)(CM_CHUNK * qs + 2 * CM_CHUNK * vs) * 2;
+    const size_t smem_o = (size_t)(2 * CM_CHUNK * qs + 2 * CM_CHUNK * vs + 2 * a->dim * vs) * 2;
     static bool opted = false;
     if (!opted) {
         RDL_CUDA(cudaFuncSetAttribute(ssc_chunk_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024), "state_space_chunked");

@@ -23,7 +23,7 @@ from concurrent.futures import ThreadPoolExecutor
 _PKG = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CSRC = os.path.join(_PKG, "csrc")
 LIB_NAME = "librdl_b200_kernels.so"
-ABI_VERSION = 20
+ABI_VERSION = 21
 
 # fast math is never enabled: the 32-bit path relies on exact tanhf/expf/sqrtf and plain FMA
 NVCC_FLAGS = ["-std=c++17", "-O3", "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo",
@@ -174,6 +174,7 @@ class AttentionArgs(ctypes.Structure):
         ("rope_cos", ctypes.c_void_p), ("rope_sin", ctypes.c_void_p), ("rotary_dim", ctypes.c_int), ("new_rows", ctypes.c_int),
         ("sinks", ctypes.c_void_p), ("sigmoid_bias", ctypes.c_void_p),
         ("chunk", ctypes.c_int), ("rel_bias", ctypes.c_void_p), ("rel_len", ctypes.c_int),
+        ("kv_share", ctypes.c_int),
         ("wait_cycles", ctypes.c_longlong), ("test_extra_tx", ctypes.c_int),     # filled in by the launcher
     ]
 
@@ -305,6 +306,70 @@ class QkvPrepareArgs(ctypes.Structure):
     ]
 
 
+class HeadPrepareArgs(ctypes.Structure):
+    """The step between a q/k/v product and attention where projections are treated head by head (`csrc/api.h`)."""
+    _fields_ = [
+        ("dtype", ctypes.c_int),
+        ("n_tokens", ctypes.c_int), ("n_seqs", ctypes.c_int),
+        ("n_heads", ctypes.c_int), ("n_kv_heads", ctypes.c_int), ("maps", ctypes.c_int),
+        ("dim", ctypes.c_int), ("vdim", ctypes.c_int), ("pad", ctypes.c_int),
+        ("rows", ctypes.c_void_p), ("row_stride", ctypes.c_longlong),
+        ("q_col", ctypes.c_int), ("k_col", ctypes.c_int), ("v_col", ctypes.c_int),
+        ("out", ctypes.c_void_p), ("out_stride", ctypes.c_longlong),
+        ("bias", ctypes.c_void_p),
+        ("conv", ctypes.c_void_p), ("taps", ctypes.c_int), ("state", ctypes.c_void_p),
+        ("wq", ctypes.c_void_p), ("wk", ctypes.c_void_p), ("eps", ctypes.c_float),
+        ("cos_t", ctypes.c_void_p), ("sin_t", ctypes.c_void_p), ("rot_n", ctypes.c_int),
+        ("q_factor", ctypes.c_void_p),
+        ("tok_pos", ctypes.c_void_p), ("seq_start", ctypes.c_void_p), ("slots", ctypes.c_void_p), ("seq_end", ctypes.c_void_p),
+        ("write_kv", ctypes.c_int), ("do_write", ctypes.c_int),
+        ("k_cache", ctypes.c_void_p), ("v_cache", ctypes.c_void_p), ("tables", ctypes.c_void_p),
+        ("table_width", ctypes.c_int), ("page_size", ctypes.c_int), ("ring_pages", ctypes.c_int),
+    ]
+
+
+class ContextSide(ctypes.Structure):
+    """One mixer's results on their way into the output product's rows (`csrc/api.h`)."""
+    _fields_ = [
+        ("x", ctypes.c_void_p), ("x_f32", ctypes.c_int), ("x_stride", ctypes.c_longlong), ("x_head", ctypes.c_int),
+        ("n_heads", ctypes.c_int), ("vdim", ctypes.c_int),
+        ("maps", ctypes.c_int), ("lam", ctypes.c_float),
+        ("norm", ctypes.c_int), ("eps", ctypes.c_float),
+        ("weight", ctypes.c_void_p), ("factor", ctypes.c_float),
+        ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_longlong), ("gate_kind", ctypes.c_int),
+        ("out_col", ctypes.c_int),
+    ]
+
+
+CONTEXT_GATES = {None: 0, "head": 1, "value": 2}
+
+
+class ContextFinishArgs(ctypes.Structure):
+    _fields_ = [
+        ("dtype", ctypes.c_int), ("n_tokens", ctypes.c_int), ("n_sides", ctypes.c_int),
+        ("side", ContextSide * 2),
+        ("out", ctypes.c_void_p), ("out_stride", ctypes.c_longlong), ("out_width", ctypes.c_int),
+        ("ones_col", ctypes.c_int), ("n_ones", ctypes.c_int),
+    ]
+
+
+class MatrixMemoryArgs(ctypes.Structure):
+    """One call of the matrix memory recurrence (`csrc/api.h`)."""
+    _fields_ = [
+        ("dtype", ctypes.c_int),
+        ("n_tokens", ctypes.c_int), ("n_seqs", ctypes.c_int), ("n_heads", ctypes.c_int), ("dim", ctypes.c_int), ("vdim", ctypes.c_int),
+        ("rows", ctypes.c_void_p), ("row_stride", ctypes.c_longlong),
+        ("q_col", ctypes.c_int), ("k_col", ctypes.c_int), ("v_col", ctypes.c_int), ("i_col", ctypes.c_int), ("f_col", ctypes.c_int),
+        ("i_bias", ctypes.c_void_p), ("f_bias", ctypes.c_void_p),
+        ("cap", ctypes.c_float), ("q_scale", ctypes.c_float), ("den_eps", ctypes.c_float),
+        ("tok_pos", ctypes.c_void_p), ("seq_start", ctypes.c_void_p), ("slots", ctypes.c_void_p),
+        ("state", ctypes.c_void_p), ("norm", ctypes.c_void_p), ("out", ctypes.c_void_p),
+    ]
+
+
+MATRIX_MEMORY_COLS = 32      # state columns that share one copy of the normaliser and the running maximum
+
+
 class HyperArgs(ctypes.Structure):
     """One step of a residual stream of several copies (`csrc/api.h`)."""
     _fields_ = [
@@ -331,7 +396,7 @@ _SIGNATURES = {
     "rdl_attention_decode": [ctypes.POINTER(AttentionArgs), _P],
     "rdl_attention_prefill_tc": [ctypes.POINTER(AttentionArgs), _LL, _P],
     "rdl_embed_rows": [_P, _P, _I, _P, _F, _I, _I, _I, _P, _P, _I, _P, _I, _P],
-    "rdl_norm_residual_norm": [_P, _I, _P, _P, _I, _F, _F, _P, _P, _I, _F, _F, _P, _I, _I, _I, _P],
+    "rdl_norm_residual_norm": [_P, _I, _P, _P, _I, _F, _F, _P, _P, _P, _P, _P, _I, _F, _F, _P, _I, _I, _I, _P],
     "rdl_gated_activation": [_P, _P, _I, _I, _I, _I, _F, _P],
     "rdl_softcap_inplace": [_P, _LL, _F, _P],
     "rdl_scale_inplace": [_P, _LL, _F, _P],
@@ -372,6 +437,11 @@ _SIGNATURES = {
     "rdl_latent_decode": [_P, _LL, _P, _LL, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _P, _LL, _P, _P],
     "rdl_moe_route": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _I, _I, _I, _F, _P],
     "rdl_qkv_prepare": [ctypes.POINTER(QkvPrepareArgs), _P],
+    "rdl_head_prepare": [ctypes.POINTER(HeadPrepareArgs), _P],
+    "rdl_context_finish": [ctypes.POINTER(ContextFinishArgs), _P],
+    "rdl_matrix_memory_scan": [ctypes.POINTER(MatrixMemoryArgs), _P],
+    "rdl_matrix_memory_copies": [_I],
+    "rdl_matrix_memory_chunked": [ctypes.POINTER(MatrixMemoryArgs), _P, _LL, _P],
     "rdl_hyper": [ctypes.POINTER(HyperArgs), _P],
     "rdl_moe_gate_up": [_P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P],
     "rdl_moe_down_combine": [_P, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
@@ -414,6 +484,8 @@ def load():
         lib.rdl_state_space_chunked_work_bytes.restype = _LL
         lib.rdl_delta_rule_chunked_work_bytes.argtypes = [_I, _I, _I, _I, _I]
         lib.rdl_delta_rule_chunked_work_bytes.restype = _LL
+        lib.rdl_matrix_memory_chunked_work_bytes.argtypes = [_I, _I, _I, _I, _I]
+        lib.rdl_matrix_memory_chunked_work_bytes.restype = _LL
         lib.rdl_latent_decode_scratch_bytes.argtypes = [_I, _I, _I, _I]
         lib.rdl_latent_decode_scratch_bytes.restype = _LL
         lib.rdl_sampling_uniform.argtypes = [ctypes.c_ulonglong] * 3

@@ -120,9 +120,13 @@ class NormParams(NamedTuple):
 
 def norm_residual_norm(x: torch.Tensor, *, first: Optional[NormParams] = None, residual: Optional[torch.Tensor] = None,
                        second: Optional[NormParams] = None, out_dtype: Optional[torch.dtype] = None,
-                       row_index: Optional[torch.Tensor] = None, want_output: bool = True):
+                       row_index: Optional[torch.Tensor] = None, want_output: bool = True,
+                       add_rows: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None,
+                       residual_out: Optional[torch.Tensor] = None):
     """t = first ? rms_norm(x; first) : x;  h = residual + t (written back to `residual`, float32)
     or t;  returns second ? rms_norm(h; second) : h in `out_dtype`, or None if not wanted.
+    add_rows (float32 [rows, hidden]) and add_vec (float32 [hidden]) are added to h as well; residual_out: where h is written
+    instead of `residual` (also without one).
     rms_norm(v; w, eps, off) = v / sqrt(mean(v^2) + eps) * (w + off), statistics in float32."""
     _dense(x, "x")
     _need(x.dim() == 2, "x must be [rows, hidden]")
@@ -136,13 +140,17 @@ def norm_residual_norm(x: torch.Tensor, *, first: Optional[NormParams] = None, r
     if residual is not None:
         _need(residual.dtype is torch.float32 and residual.is_contiguous() and tuple(residual.shape) == (rows, H),
               "residual must be a contiguous float32 [rows, hidden] tensor")
+    for t, shape, name in ((residual_out, (rows, H), "residual_out"), (add_rows, (rows, H), "add_rows"), (add_vec, (H,), "add_vec")):
+        _need(t is None or (t.dtype is torch.float32 and t.is_contiguous() and tuple(t.shape) == shape), f"norm_residual_norm: {name} must be float32 {shape}")
+    if residual_out is None:
+        residual_out = residual
     y = torch.empty((rows, H), dtype=out_dtype or x.dtype, device=x.device) if want_output else None
-    _need(y is not None or residual is not None, "norm_residual_norm: nothing to write")
+    _need(y is not None or residual_out is not None, "norm_residual_norm: nothing to write")
     library.check(library.load().rdl_norm_residual_norm(
         _ptr(x), _dtype_code(x), _ptr(row_index),
         _ptr(first.weight) if first else None, _dtype_code(first.weight) if first else 0,
         float(first.eps) if first else 0.0, float(first.offset) if first else 0.0,
-        _ptr(residual),
+        _ptr(residual), _ptr(residual_out), _ptr(add_rows), _ptr(add_vec),
         _ptr(second.weight) if second else None, _dtype_code(second.weight) if second else 0,
         float(second.eps) if second else 0.0, float(second.offset) if second else 0.0,
         _ptr(y), _dtype_code(y) if y is not None else 0, rows, H, _stream(x)))
@@ -554,7 +562,7 @@ def linear(x, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
           f"linear: activation '{activation}' is not one of {sorted(UNARY_FORMS)} (and comes without a soft-cap)")
     if isinstance(x, DeferredRows):
         _need(softcap is None or out_dtype is torch.float32, "linear: the soft-cap is applied to float32 results")
-        out = _linear_deferred(x, weight, weight.shape[0], out_dtype or x.dtype, False, 0, softcap, status) if activation is None else None
+        out = _linear_deferred(x, weight, weight.shape[0], out_dtype or x.dtype, False, UNARY_FORMS[activation] if activation else 0, softcap, status)
         if out is not None:
             return out
         x = x.materialise()
@@ -772,6 +780,118 @@ def qkv_prepare(rows: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int
     return out
 
 
+def head_prepare(rows: torch.Tensor, *, n_heads: int, n_kv_heads: int, maps: int, dim: int, vdim: int, pad: int, q_col: int, k_col: int,
+                 v_col: Optional[int], tok_pos, seq_start, slots, seq_end, n_seqs: int, bias: Optional[torch.Tensor] = None,
+                 conv: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, wq: Optional[torch.Tensor] = None,
+                 wk: Optional[torch.Tensor] = None, eps: float = 0.0, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
+                 q_factor: Optional[torch.Tensor] = None, pages: Optional[KVPages] = None, write_kv: bool = True) -> torch.Tensor:
+    """The rows of a q/k/v product made ready for attention head by head, in one pass (all in float, rounded once): bias
+    (float32 [channels of q and k]); a causal convolution over time per channel of q and k (conv: [taps, channels] in the rows'
+    dtype, row j for the value taps - 1 - j tokens back; earlier steps' values from `state`, float32 [slots, taps - 1, channels],
+    which is left holding the last ones); v_col None: the values are the keys at this point; a root-mean-square norm of every head
+    (float32 weights wq, wk [dim] for all query and all key heads); rotation of the first 2 * cos.shape[1] values of every head
+    (half-split pairs); the queries times q_factor[position]; and, with `pages`, the cache write.
+    With maps > 1 every query and key head has so many maps of `dim` values: a key head's maps lie side by side in its row, a
+    query head's map m becomes a query head of its own that is zero outside map m's columns (bias, norm and rotation are per map).
+    Returns dense rows [tokens, (n_heads * maps + 2 n_kv_heads) * pad]: heads laid out with `pad` values, zeros after their own;
+    without write_kv the key and value columns are left unwritten (the cache has them)."""
+    C = (n_heads + n_kv_heads) * maps * dim
+    _need(rows.dim() == 2 and rows.stride(1) == 1, "head_prepare: packed rows")
+    T, W = rows.shape
+    _need(q_col >= 0 and k_col >= 0 and W >= max(q_col + n_heads * maps * dim, k_col + n_kv_heads * maps * dim, 0 if v_col is None else v_col + n_kv_heads * vdim),
+          "head_prepare: the rows are narrower than the heads")
+    a = library.HeadPrepareArgs()
+    a.dtype, a.n_tokens, a.n_seqs, a.n_heads, a.n_kv_heads, a.maps = _dtype_code(rows), T, n_seqs, n_heads, n_kv_heads, maps
+    a.dim, a.vdim, a.pad = dim, vdim, pad
+    out = torch.empty((T, (n_heads * maps + 2 * n_kv_heads) * pad), dtype=rows.dtype, device=rows.device)
+    a.rows, a.row_stride, a.out, a.out_stride = rows.data_ptr(), rows.stride(0), out.data_ptr(), out.stride(0)
+    a.q_col, a.k_col, a.v_col = q_col, k_col, -1 if v_col is None else v_col
+    f32 = lambda t, n: t.dtype is torch.float32 and t.is_contiguous() and t.numel() == n
+    if bias is not None:
+        _need(f32(bias, C), f"head_prepare: the bias must be float32 [{C}]")
+        a.bias = bias.data_ptr()
+    if conv is not None:
+        _need(conv.dtype is rows.dtype and conv.is_contiguous() and conv.dim() == 2 and conv.shape[1] == C, f"head_prepare: the convolution must be [taps, {C}] in the rows' dtype")
+        taps = conv.shape[0]
+        _need(1 <= taps <= SHORT_CONV_MAX_TAPS, f"head_prepare: {taps} taps, the kernel takes 1 to {SHORT_CONV_MAX_TAPS}")
+        a.conv, a.taps = conv.data_ptr(), taps
+        if taps > 1:
+            _need(state is not None and state.dtype is torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, C),
+                  "head_prepare: the state must be float32 [slots, taps - 1, channels]")
+            a.state = state.data_ptr()
+    if wq is not None:
+        _need(f32(wq, dim) and wk is not None and f32(wk, dim), f"head_prepare: the norms' weights must be float32 [{dim}]")
+        a.wq, a.wk, a.eps = wq.data_ptr(), wk.data_ptr(), float(eps)
+    if cos is not None:
+        _need(cos.dtype is torch.float32 and sin.dtype is torch.float32 and cos.is_contiguous() and sin.is_contiguous() and cos.shape == sin.shape,
+              "rotary tables must be float32 [positions, rotated / 2]")
+        a.cos_t, a.sin_t, a.rot_n = cos.data_ptr(), sin.data_ptr(), 2 * cos.shape[1]
+    if q_factor is not None:
+        _need(q_factor.dtype is torch.float32 and q_factor.is_contiguous() and q_factor.dim() == 1, "head_prepare: the queries' factors must be float32 [positions]")
+        a.q_factor = q_factor.data_ptr()
+    _int32(tok_pos, "tok_pos", T); _int32(seq_start, "seq_start", n_seqs + 1); _int32(slots, "slots", n_seqs); _int32(seq_end, "seq_end", n_seqs)
+    a.tok_pos, a.seq_start, a.slots, a.seq_end = (t.data_ptr() for t in (tok_pos, seq_start, slots, seq_end))
+    a.write_kv = int(bool(write_kv))
+    if pages is not None:
+        _need(pages.k.dtype is rows.dtype and pages.v.dtype is rows.dtype, "cache dtype differs from the activations'")
+        _need(tuple(pages.k.shape[1:]) == (n_kv_heads, pages.page_size, pad) and pages.k.is_contiguous()
+              and pages.v.is_contiguous() and pages.v.shape == pages.k.shape, "cache storage has the wrong shape")
+        _int32(pages.tables, "page tables")
+        a.do_write = 1
+        a.k_cache, a.v_cache, a.tables, a.table_width = pages.k.data_ptr(), pages.v.data_ptr(), pages.tables.data_ptr(), pages.tables.shape[1]
+        a.page_size, a.ring_pages = pages.page_size, pages.ring_pages
+    library.check(library.load().rdl_head_prepare(ctypes.byref(a), _stream(rows)))
+    return out
+
+
+class ContextSide(NamedTuple):
+    """One mixer's results and what is still to be done with them before the output product (`context_finish`)."""
+    x: torch.Tensor                          # [tokens, n_heads * maps * head_stride], float32 or the activations' dtype
+    n_heads: int
+    vdim: int
+    head_stride: int                         # columns between heads (their laid-out size)
+    maps: int = 1                            # 2: x_1 - lam x_2
+    lam: float = 0.0
+    norm_eps: Optional[float] = None         # every head divided by its root mean square
+    weight: Optional[torch.Tensor] = None    # float32 [n_heads * vdim]
+    factor: float = 1.0
+    gate: Optional[torch.Tensor] = None      # sigmoid gate: [tokens, n_heads] or [tokens, n_heads * vdim] (a column slice of wider rows)
+    gate_kind: Optional[str] = None          # "head" or "value"
+
+
+def context_finish(sides, width: int, n_ones: int, dtype: torch.dtype) -> torch.Tensor:
+    """The output product's rows [tokens, width] from one mixer's results, or from two mixers' side by side: per side and head
+    (x_1 - lam x_2 or x), divided by its root mean square, times weight and factor, times the sigmoid of its gate, all in float
+    and rounded once; then n_ones columns of ones (for a bias that is part of the product's matrix) and zeros."""
+    _need(1 <= len(sides) <= 2, "context_finish: one or two sides")
+    T, dev = sides[0].x.shape[0], sides[0].x.device
+    out = torch.empty((T, width), dtype=dtype, device=dev)
+    a = library.ContextFinishArgs()
+    a.dtype, a.n_tokens, a.n_sides = _dtype_code(out), T, len(sides)
+    col = 0
+    for i, s in enumerate(sides):
+        _need(s.x.dim() == 2 and s.x.shape[0] == T and s.x.stride(1) == 1 and s.x.dtype in (torch.float32, dtype), "context_finish: bad results")
+        _need(s.x.shape[1] >= (s.n_heads * s.maps - 1) * s.head_stride + s.vdim, "context_finish: the results are narrower than the heads")
+        c = a.side[i]
+        c.x, c.x_f32, c.x_stride, c.x_head = s.x.data_ptr(), int(s.x.dtype is torch.float32), s.x.stride(0), s.head_stride
+        c.n_heads, c.vdim, c.maps, c.lam, c.factor, c.out_col = s.n_heads, s.vdim, s.maps, float(s.lam), float(s.factor), col
+        if s.norm_eps is not None:
+            c.norm, c.eps = 1, float(s.norm_eps)
+        if s.weight is not None:
+            _need(s.weight.dtype is torch.float32 and s.weight.is_contiguous() and s.weight.numel() == s.n_heads * s.vdim, "context_finish: the weight must be float32, one per value")
+            c.weight = s.weight.data_ptr()
+        if s.gate_kind is not None:
+            n = s.n_heads if s.gate_kind == "head" else s.n_heads * s.vdim
+            _need(s.gate.dim() == 2 and tuple(s.gate.shape) == (T, n) and s.gate.stride(1) == 1 and s.gate.dtype is dtype, f"context_finish: gates must be [tokens, {n}]")
+            c.gate, c.gate_stride = s.gate.data_ptr(), s.gate.stride(0)
+        c.gate_kind = library.CONTEXT_GATES[s.gate_kind]
+        col += s.n_heads * s.vdim
+    _need(col + n_ones <= width, f"context_finish: {col} values and {n_ones} ones in rows of {width}")
+    a.out, a.out_stride, a.out_width, a.ones_col, a.n_ones = out.data_ptr(), width, width, col, n_ones
+    library.check(library.load().rdl_context_finish(ctypes.byref(a), _stream(out)))
+    return out
+
+
 class DistanceBias(NamedTuple):
     """Numbers added to attention scores by query head and distance (query position - key position): float32 [n_heads,
     distances], the last column standing for every larger distance.  `base2` is the same table times log2(e), which the
@@ -785,6 +905,7 @@ class DistanceBias(NamedTuple):
         return DistanceBias(t, (t.to(torch.float64) * 1.4426950408889634).to(torch.float32).contiguous())
 
 
+DECODE_MAX_GROUP = 8       # query heads per key/value head a block of the decode attention kernel takes
 PREFILL_QUERY_TILE = 64    # query rows of a tile in the lists the prefill attention kernels take
 
 
@@ -927,6 +1048,13 @@ def attention(q: torch.Tensor, b: AttentionBatch, pages: Optional[KVPages], *, n
         a.keys_per_split = ks
         # a run of max_keys positions can straddle one more split than its length suggests
         a.max_splits = (max(b.max_keys, 1) + ks - 1) // ks + 1
+        group = n_heads // n_kv_heads
+        if group > DECODE_MAX_GROUP:
+            # a block takes up to eight query heads: a larger group goes to several blocks that read the same keys and values
+            share = next(s for s in range(2, group + 1) if group % s == 0 and group // s <= DECODE_MAX_GROUP)
+            n_kv_heads *= share
+            a.n_kv_heads, a.kv_share = n_kv_heads, share
+            _need(rotate_and_write is None, "attention: rotate_and_write takes groups of up to eight query heads")
         need = lib.rdl_attention_decode_scratch_bytes(b.n_tokens, n_heads, n_kv_heads, head_dim, a.max_splits)
         # the counters at the start of the scratch must be zero before a launch; the kernel leaves them so
         buf = scratch(need) if scratch is not None else torch.zeros(-(-need // 4), dtype=torch.float32, device=q.device)
@@ -1520,6 +1648,62 @@ def state_space_scan(rows: torch.Tensor, dt_rows: torch.Tensor, *, x_col: int, b
         library.check(lib.rdl_state_space_chunked(ctypes.byref(a), _ptr(work), nbytes, _stream(rows)), 3)
     else:
         raise KernelError(f"state_space_scan: unknown kind '{kind}'")
+    return out
+
+
+def matrix_memory_copies(vdim: int) -> int:
+    """Copies of the normaliser and the running maximum a head keeps (one for every so many columns of its state)."""
+    return -(-vdim // library.MATRIX_MEMORY_COLS)
+
+
+def matrix_memory_chunked_ok(rows: torch.Tensor, q_col: int, k_col: int, v_col: int, dim: int, vdim: int) -> bool:
+    """Whether the chunked kernels take these rows and sizes."""
+    return (rows.dtype is torch.bfloat16 and dim % 16 == 0 and 16 <= dim <= 128 and vdim % 16 == 0 and vdim >= 16
+            and rows.data_ptr() % 16 == 0 and rows.stride(0) % 8 == 0 and q_col % 8 == 0 and k_col % 8 == 0 and v_col % 8 == 0)
+
+
+def matrix_memory(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, i_col: int, f_col: int, n_heads: int, dim: int, vdim: int,
+                  i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, q_scale: float, den_eps: float, state: torch.Tensor,
+                  norm: torch.Tensor, tok_pos, seq_start, slots, n_seqs: int, kind: str = "auto") -> torch.Tensor:
+    """The matrix memory of xLSTM in float over the step's packed rows: per head, with i = cap tanh((rows[i_col + h] + i_bias[h]) / cap)
+    and f = log sigmoid(cap tanh((rows[f_col + h] + f_bias[h]) / cap)),
+    m_t = max(f + m_(t-1), i);  S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T;  n_t likewise with k alone;
+    o_t = S_t^T q / (max(|n_t . q|, e^(-m_t)) + den_eps), q times q_scale first.
+    state: float32 [slots, heads, dim, vdim] (S); norm: float32 [slots, heads, matrix_memory_copies(vdim), dim + 1] (n, then m
+    times log2 e; every copy alike); both are read and left holding the state after the step.  Returns float32 [tokens, heads * vdim].
+    kind: "scan" (token by token), "chunked" (bfloat16 rows, chunks of 64 tokens on tensor cores, three launches), "auto"
+    (chunks where sequences bring many tokens each)."""
+    _need(rows.dim() == 2 and rows.stride(1) == 1, "matrix_memory: packed rows")
+    T = rows.shape[0]
+    _need(min(q_col, k_col, v_col, i_col, f_col) >= 0 and rows.shape[1] >= max(q_col + n_heads * dim, k_col + n_heads * dim, v_col + n_heads * vdim, i_col + n_heads, f_col + n_heads),
+          "matrix_memory: the rows are narrower than the heads")
+    _need(state.dtype is torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (n_heads, dim, vdim), "matrix_memory: the state must be float32 [slots, heads, dim, vdim]")
+    _need(norm.dtype is torch.float32 and norm.is_contiguous() and tuple(norm.shape[1:]) == (n_heads, matrix_memory_copies(vdim), dim + 1),
+          "matrix_memory: the normaliser must be float32 [slots, heads, copies, dim + 1]")
+    _int32(tok_pos, "tok_pos", T); _int32(seq_start, "seq_start", n_seqs + 1); _int32(slots, "slots", n_seqs)
+    a = library.MatrixMemoryArgs()
+    a.dtype, a.n_tokens, a.n_seqs, a.n_heads, a.dim, a.vdim = _dtype_code(rows), T, n_seqs, n_heads, dim, vdim
+    a.rows, a.row_stride = rows.data_ptr(), rows.stride(0)
+    a.q_col, a.k_col, a.v_col, a.i_col, a.f_col = q_col, k_col, v_col, i_col, f_col
+    a.i_bias, a.f_bias = _f32_vec(i_bias, n_heads, "i_bias"), _f32_vec(f_bias, n_heads, "f_bias")
+    a.cap, a.q_scale, a.den_eps = float(cap), float(q_scale), float(den_eps)
+    a.tok_pos, a.seq_start, a.slots, a.state, a.norm = tok_pos.data_ptr(), seq_start.data_ptr(), slots.data_ptr(), state.data_ptr(), norm.data_ptr()
+    out = torch.empty((T, n_heads * vdim), dtype=torch.float32, device=rows.device)
+    a.out = out.data_ptr()
+    if kind == "auto":
+        many = T >= DECAY_CHUNKED_MIN_TOKENS and T >= DECAY_CHUNKED_MIN_PER_SEQUENCE * n_seqs
+        kind = "chunked" if (DECAY_CHUNKED and many and matrix_memory_chunked_ok(rows, q_col, k_col, v_col, dim, vdim)) else "scan"
+    lib = library.load()
+    if kind == "scan":
+        library.check(lib.rdl_matrix_memory_scan(ctypes.byref(a), _stream(rows)))
+    elif kind == "chunked":
+        _need(matrix_memory_chunked_ok(rows, q_col, k_col, v_col, dim, vdim),
+              "matrix_memory: the chunked kernels take bfloat16 rows, sizes in steps of 16 (dim up to 128) and columns on 16-byte boundaries")
+        nbytes = lib.rdl_matrix_memory_chunked_work_bytes(T, n_seqs, n_heads, dim, vdim)
+        work = torch.empty((nbytes // 4,), dtype=torch.float32, device=rows.device)
+        library.check(lib.rdl_matrix_memory_chunked(ctypes.byref(a), _ptr(work), nbytes, _stream(rows)), 3)
+    else:
+        raise KernelError(f"matrix_memory: unknown kind '{kind}'")
     return out
 
 

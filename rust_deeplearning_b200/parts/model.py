@@ -276,6 +276,11 @@ class Model:
         self.start_stream = build_part("stream", spec.stream, ctx)     # the embedded rows -> the stream the blocks work on
         self.head = build_part("head", spec.head, ctx)
         self.schedule = list(spec.schedule)
+        # what joins the stream before a run: (whether the embedded rows do, a float32 vector or None)
+        self.entries = {e: (s.enters.embedding, None if s.enters.vectors is None else
+                            ctx.tensor(s.enters.vectors)[s.enters.row].to(torch.float32).contiguous())
+                        for e, s in enumerate(self.schedule) if s.enters is not None}
+        self.keeps_embedding = any(s.enters is not None and s.enters.embedding for s in self.schedule)
         self.cache_owner_of = {e: (s.reads_cache_of if s.reads_cache_of is not None else e)
                                for e, s in enumerate(self.schedule)}
         self.shared_runs = frozenset(s.reads_cache_of for s in self.schedule if s.reads_cache_of is not None)
@@ -310,13 +315,19 @@ class Model:
         batch.new_kv.clear()
         batch.carried.clear()
         takes_positions = getattr(self.embedding, "takes_positions", False)
-        stream = self.start_stream(self.embedding.forward(batch.tokens, tok_pos=batch.tok_pos) if takes_positions
-                                   else self.embedding.forward(batch.tokens))
+        embedded = self.embedding.forward(batch.tokens, tok_pos=batch.tok_pos) if takes_positions else self.embedding.forward(batch.tokens)
+        # rows that join the stream again later stay as they are: an entry before the first run forms its sum elsewhere
+        stream = self.start_stream(embedded.clone() if self.keeps_embedding and 0 not in self.entries else embedded)
         batch.deferred_writes.clear()
         lazy_head = getattr(self.head, "takes_deferred_rows", False)
         for run, entry in enumerate(self.schedule):
             # what the stream will be asked for after this block, where the asker's first product takes the split form
-            if run + 1 < len(self.schedule):
+            if run in self.entries:
+                add, vector = self.entries[run]
+                stream.enter(embedded if add else None, vector)
+            if run + 1 in self.entries:
+                stream.norm_after_block = None
+            elif run + 1 < len(self.schedule):
                 stream.norm_after_block = getattr(self.layers[self.schedule[run + 1].layer], "first_norm", None)
             else:
                 stream.norm_after_block = self.final_norm if (lazy_head and batch.n_want) else None

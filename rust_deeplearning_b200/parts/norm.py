@@ -16,6 +16,9 @@ that reads the branch and the stream once.  Any other norm kind (anything with a
 For blocks whose sublayers all read ONE norm the stream offers `add_sum(branches, scale)`: x <- x + scale * (sum of the
 branches), formed in float32 together with the norm the next part asks for (`ops.add_branches_norm_`, one kernel).
 
+Where something joins the stream between two blocks (a loop's pass begins: `enter(rows, vector)`), it is added in the same
+kernel as the branch that still waits and the norm that is asked for next.
+
 For blocks that norm AFTER the sum the stream offers `rows(dtype)` (the stream itself as a part's input) and
 `renorm(branch, norm, alpha, dtype)`: x <- norm(alpha x + branch) in float32, in place, in one kernel that also
 leaves x in the activations' dtype for the next part.
@@ -85,6 +88,7 @@ class ResidualStream:
         self.x = x
         self._pending = None     # (branch: tensor or ops.Branch, post_norm or None)
         self._pending_sum = None     # (branches, scale): x + scale * (sum of the branches), waiting for the next norm
+        self._entering = None    # (rows or None, vector or None): joins x after the waiting branch
         self._operand = None     # (bfloat16 [16, hidden] whose first rows are x times a norm's column factors, that norm)
         self._lent = None        # DeferredRows handed out; x is valid once they have been used
         self._rows = None        # x in the activations' dtype, as `renorm` left it (valid until x changes again)
@@ -149,7 +153,34 @@ class ResidualStream:
         self._rows = None
         self._pending_sum = (tuple(b for b in branches if b is not None), float(scale))
 
+    def enter(self, rows, vector):
+        """x <- x + rows + vector (float32 [rows, hidden] and [hidden], either optional), after any waiting branch; done lazily.
+        x is then written to a buffer of its own unless a branch waits, so that rows x was built on stay as they are."""
+        self._settled()
+        if self._entering is not None:
+            self._flush()
+        self._rows = None
+        self._entering = (rows, vector)
+
+    def _enter(self, second=None, out_dtype=None):
+        """The waiting branch and what enters are added in one kernel, with the norm `second` (its rows are returned) or without."""
+        rows, vector = self._entering
+        branch, post = self._pending if self._pending is not None else (None, None)
+        if self._pending_sum is not None or isinstance(branch, ops.Branch) or not (post is None or _fusable(post)):
+            self._entering = None
+            self._flush()
+            branch = post = None
+        self._entering = self._pending = self._operand = None
+        extra = dict(add_rows=rows, add_vec=vector, second=second, want_output=second is not None, out_dtype=out_dtype)
+        if branch is not None:
+            return ops.norm_residual_norm(branch, first=post.fused_params() if post else None, residual=self.x, **extra)
+        x, self.x = self.x, torch.empty_like(self.x)
+        return ops.norm_residual_norm(x, residual_out=self.x, **extra)
+
     def _flush(self):
+        if self._entering is not None:
+            self._enter()
+            return
         if self._pending_sum is not None:
             branches, scale = self._pending_sum
             self._pending_sum = None
@@ -172,6 +203,10 @@ class ResidualStream:
         `ops.DeferredRows`.  upcoming: the norm the stream will be asked for after the next branch, if the
         caller knows it and both sides of that branch can use the split form."""
         self._settled()
+        if self._entering is not None and _fusable(norm):
+            y = self._enter(norm.fused_params(), out_dtype)
+            self._prepare(upcoming, out_dtype)
+            return y
         if self._pending_sum is not None and _fusable(norm):
             branches, scale = self._pending_sum
             self._pending_sum = None

@@ -64,12 +64,34 @@ class LayerSpec:
 
 
 @dataclass(frozen=True)
+class StreamEntry:
+    """What joins the residual stream right before a run (the start of a pass of a loop): the embedding part's rows as they
+    were before the first run (`embedding`), and row `row` of the tensor `vectors` [n, hidden], for every token alike."""
+    embedding: bool = False
+    vectors: Optional[TensorSpec] = None
+    row: int = 0
+
+
+@dataclass(frozen=True)
 class ScheduleEntry:
     """One run of a layer.  `layer` indexes `ModelSpec.layers` (a layer may be named twice:
     each run has cache storage of its own).  `reads_cache_of` names an earlier schedule entry
-    whose keys and values this run reads instead of writing its own."""
+    whose keys and values this run reads instead of writing its own.  `enters`: what joins the stream before the run."""
     layer: int
     reads_cache_of: Optional[int] = None
+    enters: Optional[StreamEntry] = None
+
+
+def looped_schedule(n_layers: int, start: int, stop: int, times: int, vectors: Optional[TensorSpec] = None) -> Tuple[ScheduleEntry, ...]:
+    """Layers 0 .. n_layers - 1 in order, of which start .. stop - 1 run `times` times in a row (each pass with cache storage of
+    its own).  Before every pass but the first the embedded rows join the stream, and before every pass its row of `vectors`."""
+    if not (0 <= start < stop <= n_layers and times >= 1):
+        raise ValueError(f"a loop of layers {start} to {stop - 1}, {times} times, does not fit {n_layers} layers")
+    out = [ScheduleEntry(i) for i in range(start)]
+    for t in range(times):
+        enters = StreamEntry(t > 0, vectors, t) if (t > 0 or vectors is not None) else None
+        out += [ScheduleEntry(i, None, enters if i == start else None) for i in range(start, stop)]
+    return tuple(out + [ScheduleEntry(i) for i in range(stop, n_layers)])
 
 
 @dataclass(frozen=True)
@@ -101,6 +123,8 @@ class ModelSpec:
                 yield n
             if layer.tensors:
                 yield PartSpec("block_tensors", {}, layer.tensors)
+        for v in {e.enters.vectors for e in self.schedule if e.enters is not None and e.enters.vectors is not None}:
+            yield PartSpec("entry_vectors", {}, {"vectors": v})
         yield self.final_norm
         yield self.head
 
@@ -120,6 +144,9 @@ class ModelSpec:
         for e, entry in enumerate(self.schedule):
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(f"schedule entry {e} names layer {entry.layer}, model has {len(self.layers)}")
+            v = entry.enters.vectors if entry.enters is not None else None
+            if v is not None and (len(v.shape) != 2 or not 0 <= entry.enters.row < v.shape[0]):
+                raise ValueError(f"schedule entry {e} takes row {entry.enters.row} of '{v.name}', which has the shape {v.shape}")
             if entry.reads_cache_of is not None and not 0 <= entry.reads_cache_of < e:
                 raise ValueError(f"schedule entry {e} reads the cache of entry {entry.reads_cache_of}, "
                                  f"which does not run before it")
