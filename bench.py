@@ -327,6 +327,26 @@ def gasetar_window_shape(width, heads, kv_heads, dim, window, experts, top, ff, 
             "layers": [{"type": "attention", "mixer": attn, "mlp": moe if i % 2 else {"kind": "dense", "ff": dense_ff}} for i in range(layers)]}
 
 
+def paditar_shape(width, heads, kv_heads, dim, ff, vocab, times=2):
+    """A Paditar configuration of four layers - two pairs (attention beside a matrix memory) that run `times` times, differential
+    attention (two maps of half a head each), a pair - each with a dense feed-forward."""
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "conv": 4, "q_temp": {"coef": 0.1, "every": 4096}}
+    pair = {"type": "parallel", "mixer": {"left": left, "right": {"heads": heads, "dim": dim, "vdim": dim, "gate_cap": 15.0}, "left_scale": 0.7, "right_scale": 0.7}}
+    diff = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "scale": (dim // 2) ** -0.5,
+                                           "diff": 0.3, "rot": {"base": 1e4, "dims": dim // 2}}}
+    return {"architecture": "Paditar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 2, "times": times},
+            "max_positions": CONTEXT, "layers": [dict(l, mlp={"kind": "dense", "ff": ff}) for l in (pair, pair, diff, pair)]}
+
+
+def dokulorn_pairs_shape(width, heads, kv_heads, dim, ff, vocab, times=2):
+    """The Dokulorn configuration with as many layers as a Paditar one runs: pairs (softmax attention beside lightning attention)
+    where that one has pairs, a retention layer where it has differential attention."""
+    cfg = dokulorn_shape(width, heads, kv_heads, dim, ff, 4, vocab)
+    ret, pair = cfg["layers"][0], cfg["layers"][3]
+    cfg["layers"] = [pair] * (2 * times) + [ret, pair]
+    return cfg
+
+
 DESIGN_SIZES = {
     # name: (the design's arguments, the Gemma 2 arguments of equal width / heads / active feed-forward width)
     "w1024": (dict(width=1024, heads=8, dim=64, rot_dim=64, vdim=128, kv_rank=192, window=1024, experts=16, identity=2, top=2, ff=1024,
@@ -376,6 +396,15 @@ KITONEX_SIZES = {
                    shared_ff=2304, dense_ff=8448, vocab=32000),
               dict(width=2048, heads=16, kv_heads=8, dim=128, window=4096, experts=64, top=6, ff=1024, shared_ff=2304, dense_ff=8448, vocab=32000)),
 }
+PADITAR_SIZES = {
+    # four layers, six runs; Dokulorn, the closest registered design (softmax attention beside a recurrence with a state of fixed
+    # size in one layer), with six layers, the same width, heads, key heads and head size, and feed-forwards of equal size
+    # (three matrices of two thirds the width)
+    "w1024": (dict(width=1024, heads=8, kv_heads=4, dim=128, ff=4608, vocab=32000),
+              dict(width=1024, heads=8, kv_heads=4, dim=128, ff=3072, vocab=32000)),
+    "w2048": (dict(width=2048, heads=16, kv_heads=8, dim=128, ff=9216, vocab=32000),
+              dict(width=2048, heads=16, kv_heads=8, dim=128, ff=6144, vocab=32000)),
+}
 # design -> (its shape, its sizes, the title, the registered design it stands beside and that design's shape)
 DESIGNS = {"ligirax": (ligirax_shape, DESIGN_SIZES, "ligirax beside gemma2 at equal width, heads and active feed-forward width", "gemma2", gemma_like),
            "dokulorn": (dokulorn_shape, DOKULORN_SIZES, "dokulorn beside gemma2 at equal width, heads, head size and feed-forward width", "gemma2",
@@ -384,6 +413,8 @@ DESIGNS = {"ligirax": (ligirax_shape, DESIGN_SIZES, "ligirax beside gemma2 at eq
                        "gemma2", gemma_like),
            "kitonex": (kitonex_shape, KITONEX_SIZES, "kitonex beside gasetar at equal width, heads, key heads, head size, window (chunk), experts and feed-forward widths",
                        "gasetar", gasetar_window_shape),
+           "paditar": (paditar_shape, PADITAR_SIZES, "paditar beside dokulorn at equal runs, width, heads, key heads, head size and feed-forward size",
+                       "dokulorn", dokulorn_pairs_shape),
            "revepel": (revepel_shape, REVEPEL_SIZES, "revepel beside dokulorn at equal width, heads, head size and active feed-forward width",
                        "dokulorn", dokulorn_shape)}
 
@@ -476,7 +507,7 @@ def main():
     ap.add_argument("--batch", type=int, default=8, help="batch of the --only decode case")
     ap.add_argument("--context", type=int, default=PROMPT, help="prompt length of the --only decode case")
     ap.add_argument("--no-large", action="store_true", help="leave out the 9B and 27B shapes and the long contexts")
-    ap.add_argument("--design", choices=["ligirax", "dokulorn", "revepel", "gasetar", "kitonex"], default=None,
+    ap.add_argument("--design", choices=["ligirax", "dokulorn", "revepel", "gasetar", "kitonex", "paditar"], default=None,
                     help="instead of the default workload: prefill and decode of this design beside its closest registered design "
                          "(Gemma 2; for revepel, Dokulorn; for kitonex, Gasetar) at equal layer sizes")
     ap.add_argument("--size", default=None, help="with --design: one of the sizes only")

@@ -7,7 +7,8 @@
 //   o = o * sigmoid(gate)               a gate per head or per value (optional)
 // rounded once into the side's columns of the output rows.  Columns that carry the output product's bias (`ones`) are set to
 // one, the columns after them up to the rows' width to zero.
-// A warp takes one head of one token; the order of its sums depends on the head's size alone.
+// A team of LANES lanes takes one head of one token, in pieces of 16 bytes of the result where sizes and addresses allow; the order
+// of its sums depends on the head's size alone.
 #include "api.h"
 #include "common.cuh"
 #include "launch.cuh"
@@ -21,13 +22,18 @@ template <int VEC> __device__ __forceinline__ void cf_load(const void* p, long l
     if constexpr (VEC == 1) {
         f[0] = rdl_load(p, i, dtype);
     } else if (dtype == RDL_BF16) {
-        const uint2 raw = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p + i);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-        f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+        if constexpr (VEC == 8) {
+            const uint4 raw = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p + i);
+            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { const float2 v = __bfloat1622float2(h[k]); f[2 * k] = v.x; f[2 * k + 1] = v.y; }
+        }
     } else {
-        const float4 v = *reinterpret_cast<const float4*>((const float*)p + i);
-        f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+#pragma unroll
+        for (int k = 0; k < VEC; k += 4) {
+            const float4 v = *reinterpret_cast<const float4*>((const float*)p + i + k);
+            f[k] = v.x; f[k + 1] = v.y; f[k + 2] = v.z; f[k + 3] = v.w;
+        }
     }
 }
 template <typename T, int VEC> __device__ __forceinline__ void cf_store(T* p, const float (&f)[VEC]) {
@@ -36,11 +42,11 @@ template <typename T, int VEC> __device__ __forceinline__ void cf_store(T* p, co
     } else if constexpr (sizeof(T) == 4) {
         *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
     } else {
-        const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
-        uint2 raw;
-        raw.x = *reinterpret_cast<const uint32_t*>(&a);
-        raw.y = *reinterpret_cast<const uint32_t*>(&b);
-        *reinterpret_cast<uint2*>(p) = raw;
+        uint4 raw;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) h[k] = __floats2bfloat162_rn(f[2 * k], f[2 * k + 1]);
+        *reinterpret_cast<uint4*>(p) = raw;
     }
 }
 // results that are rounded to bfloat16 take the hardware's exponential and reciprocal
@@ -48,18 +54,17 @@ template <typename T> __device__ __forceinline__ float cf_sigmoid(float z) {
     return sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(fminf(-z, 80.0f))) : 1.0f / (1.0f + expf(-z));
 }
 
-template <typename T, int VEC, int NP>
+template <typename T, int VEC, int NP, int LANES>
 __global__ void __launch_bounds__(CF_WARPS * 32) context_finish_kernel(ContextFinishArgs a) {
     rdl_grid_wait();
     rdl_grid_launch_dependents();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int heads0 = a.side[0].n_heads, heads = heads0 + (a.n_sides > 1 ? a.side[1].n_heads : 0);
-    const long long item = (long long)blockIdx.x * CF_WARPS + warp;
-    if (item >= (long long)a.n_tokens * heads) return;
-    const int t = (int)(item / heads), hh = (int)(item - (long long)t * heads);
-    const bool second = hh >= heads0;
-    const ContextSide& s = a.side[second ? 1 : 0];
-    const int h = second ? hh - heads0 : hh;
+    constexpr int TEAMS = CF_WARPS * 32 / LANES;
+    const int team = threadIdx.x / LANES, lane = threadIdx.x % LANES;
+    const unsigned mask = LANES == 32 ? 0xffffffffu : ((1u << (LANES & 31)) - 1u) << ((threadIdx.x & 31) / LANES * LANES);
+    const ContextSide& s = a.side[blockIdx.y];
+    const long long item = (long long)blockIdx.x * TEAMS + team;
+    if (item >= (long long)a.n_tokens * s.n_heads) return;
+    const int t = (int)(item / s.n_heads), h = (int)(item - (long long)t * s.n_heads);
     T* out = (T*)a.out + (long long)t * a.out_stride;
     const int x_dtype = s.x_f32 ? RDL_F32 : a.dtype;
     const long long x0 = (long long)t * s.x_stride + (long long)h * s.maps * s.x_head;
@@ -67,7 +72,7 @@ __global__ void __launch_bounds__(CF_WARPS * 32) context_finish_kernel(ContextFi
     float v[NP][VEC], x2[NP][VEC], gv[NP][VEC], wv[NP][VEC];
 #pragma unroll
     for (int p = 0; p < NP; ++p) {
-        const int e = (p * 32 + lane) * VEC;
+        const int e = (p * LANES + lane) * VEC;
 #pragma unroll
         for (int i = 0; i < VEC; ++i) { v[p][i] = 0.f; x2[p][i] = 0.f; gv[p][i] = 0.f; wv[p][i] = 1.f; }
         if (e < s.vdim) {
@@ -90,13 +95,14 @@ __global__ void __launch_bounds__(CF_WARPS * 32) context_finish_kernel(ContextFi
         for (int p = 0; p < NP; ++p)
 #pragma unroll
             for (int i = 0; i < VEC; ++i) ss = fmaf(v[p][i], v[p][i], ss);
-        ss = warp_sum(ss);
+#pragma unroll
+        for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
         inv *= 1.0f / sqrtf(ss / (float)s.vdim + s.eps);
     }
     if (s.gate_kind == RDL_CONTEXT_GATE_HEAD) inv *= cf_sigmoid<T>(one_gate);
 #pragma unroll
     for (int p = 0; p < NP; ++p) {
-        const int e = (p * 32 + lane) * VEC;
+        const int e = (p * LANES + lane) * VEC;
         if (e >= s.vdim) continue;
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
@@ -106,20 +112,27 @@ __global__ void __launch_bounds__(CF_WARPS * 32) context_finish_kernel(ContextFi
         }
         cf_store<T, VEC>(out + s.out_col + h * s.vdim + e, v[p]);
     }
-    if (hh == heads - 1)
-        for (int c = a.ones_col + lane; c < a.out_width; c += 32) out[c] = from_float<T>(c < a.ones_col + a.n_ones ? 1.f : 0.f);
+    if (blockIdx.y == 0 && h == 0)
+        for (int c = a.ones_col + lane; c < a.out_width; c += LANES) out[c] = from_float<T>(c < a.ones_col + a.n_ones ? 1.f : 0.f);
 }
 
+template <typename T, int VEC, int NP, int LANES>
+cudaError_t launch_as(const ContextFinishArgs& a, long long items, cudaStream_t st) {
+    constexpr int TEAMS = CF_WARPS * 32 / LANES;
+    return rdl_launch(context_finish_kernel<T, VEC, NP, LANES>, dim3((unsigned)((items + TEAMS - 1) / TEAMS), a.n_sides), dim3(CF_WARPS * 32), 0, st, a);
+}
+
+// items: heads of the side that has most, over all tokens
 template <typename T>
-cudaError_t launch_finish(const ContextFinishArgs& a, bool vec, int widest, long long items, cudaStream_t st) {
-    const dim3 grid((unsigned)((items + CF_WARPS - 1) / CF_WARPS)), block(CF_WARPS * 32);
-    if (vec) {
-        if (widest <= 128) return rdl_launch(context_finish_kernel<T, 4, 1>, grid, block, 0, st, a);
-        if (widest <= 256) return rdl_launch(context_finish_kernel<T, 4, 2>, grid, block, 0, st, a);
-        return rdl_launch(context_finish_kernel<T, 4, 4>, grid, block, 0, st, a);
+cudaError_t launch_finish(const ContextFinishArgs& a, bool wide, int widest, long long items, cudaStream_t st) {
+    constexpr int VEC = 16 / (int)sizeof(T);
+    if (wide) {
+        if (widest <= 8 * VEC) return launch_as<T, VEC, 1, 8>(a, items, st);
+        if (widest <= 16 * VEC) return launch_as<T, VEC, 1, 16>(a, items, st);
+        if (widest <= 32 * VEC) return launch_as<T, VEC, 1, 32>(a, items, st);
+        return launch_as<T, VEC, CF_MAX_DIM / (32 * VEC), 32>(a, items, st);
     }
-    if (widest <= 128) return rdl_launch(context_finish_kernel<T, 1, 4>, grid, block, 0, st, a);
-    return rdl_launch(context_finish_kernel<T, 1, 16>, grid, block, 0, st, a);
+    return widest <= 128 ? launch_as<T, 1, 4, 32>(a, items, st) : launch_as<T, 1, 16, 32>(a, items, st);
 }
 
 }  // namespace
@@ -128,9 +141,9 @@ extern "C" int rdl_context_finish(const ContextFinishArgs* p, void* stream) {
     const ContextFinishArgs& a = *p;
     RDL_REQUIRE(rdl_valid_dtype(a.dtype) && a.n_tokens >= 0 && (a.n_sides == 1 || a.n_sides == 2) && a.out, "context_finish: bad arguments");
     const int es = a.dtype == RDL_BF16 ? 2 : 4;
-    bool vec = a.out_stride % 4 == 0 && ((uintptr_t)a.out & 15) == 0;
-    int widest = 0, used = 0;
-    long long heads = 0;
+    const int per = 16 / es;                    // values of a 16-byte piece of the result
+    bool wide = a.out_stride % per == 0 && ((uintptr_t)a.out & 15) == 0;
+    int widest = 0, used = 0, heads = 0;
     for (int i = 0; i < a.n_sides; ++i) {
         const ContextSide& s = a.side[i];
         RDL_REQUIRE(s.x && s.n_heads > 0 && s.vdim > 0 && s.vdim <= CF_MAX_DIM && (s.maps == 1 || s.maps == 2) && s.x_head >= s.vdim,
@@ -141,17 +154,16 @@ extern "C" int rdl_context_finish(const ContextFinishArgs* p, void* stream) {
         RDL_REQUIRE(s.out_col >= used && s.out_col + (long long)s.n_heads * s.vdim <= a.out_width, "context_finish: the sides' columns overlap or leave the rows");
         used = s.out_col + s.n_heads * s.vdim;
         if (s.vdim > widest) widest = s.vdim;
-        heads += s.n_heads;
-        const int xs = s.x_f32 ? 4 : es;
-        vec = vec && s.vdim % 4 == 0 && s.x_head % 4 == 0 && s.x_stride % 4 == 0 && s.out_col % 4 == 0 && ((uintptr_t)s.x & (4 * xs - 1)) == 0 &&
-              (s.gate_kind != RDL_CONTEXT_GATE_VALUE || (s.gate_stride % 4 == 0 && ((uintptr_t)s.gate & (4 * es - 1)) == 0)) && ((uintptr_t)s.weight & 15) == 0;
+        if (s.n_heads > heads) heads = s.n_heads;
+        wide = wide && s.vdim % per == 0 && s.x_head % per == 0 && s.x_stride % per == 0 && s.out_col % per == 0 && ((uintptr_t)s.x & 15) == 0 &&
+               (s.gate_kind != RDL_CONTEXT_GATE_VALUE || (s.gate_stride % per == 0 && ((uintptr_t)s.gate & 15) == 0)) && ((uintptr_t)s.weight & 15) == 0;
     }
     RDL_REQUIRE(a.ones_col >= used && a.n_ones >= 0 && a.ones_col + a.n_ones <= a.out_width && a.out_width <= a.out_stride, "context_finish: bad columns of ones");
     if (a.n_tokens == 0) return 0;
-    const long long items = heads * a.n_tokens;
+    const long long items = (long long)heads * a.n_tokens;
     RDL_REQUIRE(items / CF_WARPS < 2147483647LL, "context_finish: too many heads for one grid");
     cudaStream_t st = (cudaStream_t)stream;
-    cudaError_t e = a.dtype == RDL_BF16 ? launch_finish<__nv_bfloat16>(a, vec, widest, items, st) : launch_finish<float>(a, vec, widest, items, st);
+    cudaError_t e = a.dtype == RDL_BF16 ? launch_finish<__nv_bfloat16>(a, wide, widest, items, st) : launch_finish<float>(a, wide, widest, items, st);
     RDL_CHECK_EX(e, "context_finish");
     return 0;
 }
