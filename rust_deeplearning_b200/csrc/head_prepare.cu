@@ -193,6 +193,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prepare_kernel(HeadPrepare
             if (is_q ? (e < at_ || e >= at_ + width) : e >= at_ + width)
                 hp_store<T, VEC>(dst + (swizzle_row < 0 ? e : rdl_cache_col<T>(swizzle_row, e, D)), zero);
     };
+    const float inv_dim = 1.0f / (float)a.dim;
     const bool k_others = is_q ? width < D : (map == a.maps - 1 && at + width < D);
     const bool v_others = (is_v ? v0 + width == a.vdim : true) && a.vdim < D;
     for (int rb = r0; rb < end; rb += NT) {
@@ -251,7 +252,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prepare_kernel(HeadPrepare
                     for (int e = 0; e < VEC; ++e) ss = fmaf(v[p][e], v[p][e], ss);
 #pragma unroll
                 for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
-                const float mean = ss / (float)a.dim + a.eps;
+                const float mean = fmaf(ss, inv_dim, a.eps);
                 const float inv = sizeof(T) == 2 ? rsqrtf(mean) : 1.0f / sqrtf(mean);
 #pragma unroll
                 for (int p = 0; p < NP; ++p)
@@ -336,7 +337,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prepare_kernel(HeadPrepare
 template <typename T, int VEC, int NP, int LANES, int TAPS>
 cudaError_t launch_taps(const HeadPrepareArgs& a, cudaStream_t st) {
     constexpr int SPAN = LANES * VEC * NP, TEAMS = HP_WARPS * 32 / LANES;
-    constexpr int NT = VEC * NP <= 4 ? 4 : (VEC * NP <= 8 ? 2 : 1);          // as many tokens as a lane's registers hold
+    constexpr int NT = VEC * NP <= 4 ? 4 : 1;          // as many tokens as a lane's registers hold
     const int items = (a.n_heads + a.n_kv_heads) * a.maps + (a.v_col >= 0 ? a.n_kv_heads * ((a.vdim + SPAN - 1) / SPAN) : 0);
     const unsigned gy = (unsigned)((items + TEAMS - 1) / TEAMS);
     if (a.n_tokens <= a.n_seqs) return rdl_launch(head_prepare_kernel<T, VEC, NP, LANES, 1, TAPS, true>, dim3(a.n_seqs, gy), dim3(HP_WARPS * 32), 0, st, a);
