@@ -1,6 +1,6 @@
 """Paditar: typed configuration and its description as parts.
 
-A decoder-only model of layers listed one by one in config.json, of which a stretch runs several times in a row with the same
+A decoder-only model of layers listed one by one in config.json, of which a stretch is a loop of several passes over the same
 weights (`loop`: layers `start` to `stop` - 1, `times` passes, each with its own cache and state).  Before every pass but the
 first the embedded tokens join the residual stream again, and before every pass a learned vector of that pass does
 (`loop.step`).  Every sublayer has a norm before and a norm after it, x <- x + norm'(f(norm(x))), scale-only root-mean-square

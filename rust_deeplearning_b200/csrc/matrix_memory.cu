@@ -1,7 +1,7 @@
 // The matrix memory of xLSTM: per sequence and head a float state S [dim][vdim], a normaliser n [dim] and a running
 // maximum m, with a log input gate i and a log forget gate f per head and token,
 //   i = cap tanh((x_i + b_i) / cap),   f = log sigmoid(cap tanh((x_f + b_f) / cap)),
-//   m_t = max(f + m_(t-1), i),   S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T,   n_t likewise with k alone,
+//   m_t = max(f + m_(t-1), i),   S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T,   n_t by the same rule with k for k v^T,
 //   o = S_t^T q / (max(|n_t . q|, e^(-m_t)) + den_eps),     S, n and m zero before the first token,
 // where q is multiplied by q_scale first.  Everything but the projections (the rows) is float.  Logarithms are kept to base
 // two (m in the state too), so that every exponential is a power of two.

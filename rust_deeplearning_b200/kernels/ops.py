@@ -1667,7 +1667,7 @@ def matrix_memory(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, i_c
                   norm: torch.Tensor, tok_pos, seq_start, slots, n_seqs: int, kind: str = "auto") -> torch.Tensor:
     """The matrix memory of xLSTM in float over the step's packed rows: per head, with i = cap tanh((rows[i_col + h] + i_bias[h]) / cap)
     and f = log sigmoid(cap tanh((rows[f_col + h] + f_bias[h]) / cap)),
-    m_t = max(f + m_(t-1), i);  S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T;  n_t likewise with k alone;
+    m_t = max(f + m_(t-1), i);  S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T;  n_t by the same rule with k for k v^T;
     o_t = S_t^T q / (max(|n_t . q|, e^(-m_t)) + den_eps), q times q_scale first.
     state: float32 [slots, heads, dim, vdim] (S); norm: float32 [slots, heads, matrix_memory_copies(vdim), dim + 1] (n, then m
     times log2 e; every copy alike); both are read and left holding the state after the step.  Returns float32 [tokens, heads * vdim].

@@ -14,9 +14,9 @@ attention kernel done in one pass (`ops.head_prepare`) and what lies between att
   q_temperature  {"coef", "every"}: q is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p
   off_by_one     one joins the softmax's denominator: a sink whose logit is 0, for every head
   differential   {"diff", "eps"}: differential attention ("Differential Transformer", Ye et al.).  Every query and key head has
-                 two maps of head_dim values, each with a softmax of its own over the same values;
+                 two maps of head_dim values: two softmaxes that weight one set of values;
                  o = a_1 - lambda a_2, lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (tensor roles "lq1", "lk1", "lq2", "lk2"
-                 [head_dim]; one number for the layer); o is divided by its root mean square and multiplied by 1 - diff
+                 [head_dim], all heads share it); every head of o is normed to a root mean square of 1 - diff
   gate           "value": the concatenated heads are multiplied element by element by sigmoid(W_g x) before W_o;
                  "head": every head by one number, sigmoid(W_g x)_h
   value_dim      values of another size than keys

@@ -3,7 +3,7 @@
 Per head, over a sequence's tokens (S [dim, vdim], n [dim] and m start at zero):
     i = cap tanh((W_i x + b_i) / cap),   f = log sigmoid(cap tanh((W_f x + b_f) / cap))
     m_t = max(f + m_(t-1), i)
-    S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T,      n_t likewise with k alone
+    S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v^T,      n_t by the same rule with k for k v^T
     o_t = S_t^T (q_scale q) / (max(|n_t . q_scale q|, e^(-m_t)) + den_eps)
 Every head's o is divided by its root mean square; the concatenated heads are multiplied by the weight `norm` and by
 sigmoid(W_g x), element by element, before W_o.  The cap, q's scale, den_eps and the norm's eps are parameters.

@@ -83,7 +83,7 @@ class ScheduleEntry:
 
 
 def looped_schedule(n_layers: int, start: int, stop: int, times: int, vectors: Optional[TensorSpec] = None) -> Tuple[ScheduleEntry, ...]:
-    """Layers 0 .. n_layers - 1 in order, of which start .. stop - 1 run `times` times in a row (each pass with cache storage of
+    """Layers 0 .. n_layers - 1 in order, start .. stop - 1 of them as a loop of `times` passes (cache storage for each pass of
     its own).  Before every pass but the first the embedded rows join the stream, and before every pass its row of `vectors`."""
     if not (0 <= start < stop <= n_layers and times >= 1):
         raise ValueError(f"a loop of layers {start} to {stop - 1}, {times} times, does not fit {n_layers} layers")
